@@ -36,70 +36,84 @@ __global__ void __launch_bounds__(WARPS * 32) attention_rows_kernel(const RowsAr
     const int dk = a.d0 + a.d1, dv = a.dv;
     const float slope = a.slopes ? a.slopes[h] : 0.f;
 
-    const T* qp = a.q0 + (long long)t * a.q0_token + (long long)h * a.q0_head;
-    for (int d = lane; d < a.d0; d += 32) q_s[warp][d] = to_float(qp[d]);
-    if (a.d1 > 0) {
-        const T* qr = a.q1 + (long long)t * a.q1_token + (long long)h * a.q1_head;
-        for (int d = lane; d < a.d1; d += 32) q_s[warp][a.d0 + d] = to_float(qr[d]);
-    }
-    __syncwarp();
-
     const int* table = a.page_table + (size_t)r * a.table_width;
     constexpr int ACC = MAX_DV / 32;
-    float acc[ACC];
+    float first[ACC];  // with two maps a head: what the first map's softmax gave
 #pragma unroll
-    for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
-    // a sink stands for a key of score sinks[h] and no value: the running maximum and sum start from it
-    float m = a.sinks ? a.sinks[h] : -INFINITY, l = a.sinks ? 1.f : 0.f;
-
-    const int c_lo = (lo / 32) * 32, c_kept = ((kept + 31) / 32) * 32;  // the chunks of the kept keys end before c_kept
-    for (int c = kept > 0 ? 0 : c_lo; c <= pos; c += 32) {
-        if (c >= c_kept && c < c_lo) c = c_lo;  // nothing is seen between the kept keys and the window
-        const int j = c + lane;
-        const bool visible = (j >= lo && j <= pos) || j < kept;
-        float s = -INFINITY;
-        if (visible) {
-            const int page = table[j / a.page_size], off = j % a.page_size;
-            const T* kp = a.keys + (long long)page * a.k_page + (long long)kvh * a.k_head + (long long)off * a.k_token;
-            float dot = 0.f;
-            for (int d = 0; d < dk; ++d) dot = fmaf(q_s[warp][d], to_float(kp[d]), dot);
-            s = dot * a.scale;
-            if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
-            s -= slope * (float)(pos - j);
+    for (int i = 0; i < ACC; ++i) first[i] = 0.f;
+    for (int map = 0; map < a.maps; ++map) {
+        const T* qp = a.q0 + (long long)t * a.q0_token + (long long)h * a.q0_head + map * a.q_map;
+        __syncwarp();
+        for (int d = lane; d < a.d0; d += 32) q_s[warp][d] = to_float(qp[d]);
+        if (a.d1 > 0) {
+            const T* qr = a.q1 + (long long)t * a.q1_token + (long long)h * a.q1_head;
+            for (int d = lane; d < a.d1; d += 32) q_s[warp][a.d0 + d] = to_float(qr[d]);
         }
-        const float m_new = fmaxf(m, warp_max(s));  // finite: the chunk holds at least one visible key
-        const float p = visible ? expf(s - m_new) : 0.f;
-        const float rescale = expf(m - m_new);  // 0 on the first chunk (m = -inf)
-        l = l * rescale + warp_sum(p);
+        __syncwarp();
+
+        float acc[ACC];
 #pragma unroll
-        for (int i = 0; i < ACC; ++i) acc[i] *= rescale;
-        m = m_new;
-        const int count = min(32, pos - c + 1);
-        for (int jj = 0; jj < count; ++jj) {
-            const float pj = __shfl_sync(0xffffffffu, p, jj);
-            if (pj == 0.f) continue;  // uniform across the warp
-            const int key = c + jj;
-            const int page = table[key / a.page_size], off = key % a.page_size;
-            const T* vp = a.values + (long long)page * a.v_page + (long long)kvh * a.v_head + (long long)off * a.v_token;
+        for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
+        // a sink stands for a key of score sinks[h] and no value: the running maximum and sum start from it
+        float m = a.sinks ? a.sinks[h] : -INFINITY, l = a.sinks ? 1.f : 0.f;
+
+        const int c_lo = (lo / 32) * 32, c_kept = ((kept + 31) / 32) * 32;  // the chunks of the kept keys end before c_kept
+        for (int c = kept > 0 ? 0 : c_lo; c <= pos; c += 32) {
+            if (c >= c_kept && c < c_lo) c = c_lo;  // nothing is seen between the kept keys and the window
+            const int j = c + lane;
+            const bool visible = (j >= lo && j <= pos) || j < kept;
+            float s = -INFINITY;
+            if (visible) {
+                const int page = table[j / a.page_size], off = j % a.page_size;
+                const T* kp = a.keys + (long long)page * a.k_page + (long long)kvh * a.k_head + (long long)off * a.k_token + map * a.k_map;
+                float dot = 0.f;
+                for (int d = 0; d < dk; ++d) dot = fmaf(q_s[warp][d], to_float(kp[d]), dot);
+                s = dot * a.scale;
+                if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+                s -= slope * (float)(pos - j);
+            }
+            const float m_new = fmaxf(m, warp_max(s));  // finite: the chunk holds at least one visible key
+            const float p = visible ? expf(s - m_new) : 0.f;
+            const float rescale = expf(m - m_new);  // 0 on the first chunk (m = -inf)
+            l = l * rescale + warp_sum(p);
 #pragma unroll
-            for (int i = 0; i < ACC; ++i) {
-                const int d = lane + 32 * i;
-                if (d < dv) acc[i] = fmaf(pj, to_float(vp[d]), acc[i]);
+            for (int i = 0; i < ACC; ++i) acc[i] *= rescale;
+            m = m_new;
+            const int count = min(32, pos - c + 1);
+            for (int jj = 0; jj < count; ++jj) {
+                const float pj = __shfl_sync(0xffffffffu, p, jj);
+                if (pj == 0.f) continue;  // uniform across the warp
+                const int key = c + jj;
+                const int page = table[key / a.page_size], off = key % a.page_size;
+                const T* vp = a.values + (long long)page * a.v_page + (long long)kvh * a.v_head + (long long)off * a.v_token;
+#pragma unroll
+                for (int i = 0; i < ACC; ++i) {
+                    const int d = lane + 32 * i;
+                    if (d < dv) acc[i] = fmaf(pj, to_float(vp[d]), acc[i]);
+                }
             }
         }
-    }
-    const float inv = 1.f / l;
-    T* op = a.out + (long long)t * a.out_token + (long long)h * a.out_head;
-    const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (long long)h * dv : nullptr;
+        const float inv = 1.f / l;
 #pragma unroll
-    for (int i = 0; i < ACC; ++i) {
-        const int d = lane + 32 * i;
-        if (d < dv) {
-            float y = acc[i] * inv;
-            if (gp) y *= 1.f / (1.f + expf(-gp[d]));
-            op[d] = from_float<T>(y);
-        }
+        for (int i = 0; i < ACC; ++i) first[i] = map == 0 ? acc[i] * inv : first[i] - a.diff_weight * (acc[i] * inv);
     }
+    if (a.maps == 2) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < ACC; ++i) ss = fmaf(first[i], first[i], ss);  // lanes beyond dv hold zeros
+        const float norm = a.diff_scale / sqrtf(warp_sum(ss) / (float)dv + a.diff_eps);
+#pragma unroll
+        for (int i = 0; i < ACC; ++i) first[i] *= norm;
+    }
+    float* y = q_s[warp];  // the queries have been read
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < ACC; ++i)
+        if (lane + 32 * i < dv) y[lane + 32 * i] = first[i];
+    __syncwarp();
+    const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (a.gate_per_head ? (long long)h : (long long)h * dv) : nullptr;
+    write_head<T>(y, dv, lane, a.turn ? a.turn + (size_t)t * (dv >> 1) : nullptr, a.turn_neighbours, gp, a.gate_per_head ? 0 : 1,
+                  a.out + (long long)t * a.out_token + (long long)h * a.out_head);
 }
 
 template <typename T>
@@ -114,7 +128,8 @@ int launch_rows(const RowsArgs<T>& a, cudaStream_t stream) {
 }  // namespace
 
 // Queries in two runs of lanes, keys and values by strides, an optional distance bias per head: the form that
-// attention with other key than value sizes, and attention over a latent that is key and value at once, come in.
+// attention with other key than value sizes, attention over a latent that is key and value at once, and heads of two score
+// maps come in.  turn: [n_tokens, dv / 2] pairs (cos, sin) or null.
 LLM_EXPORT int llm_attention_rows(const void* q0, long long q0_token, long long q0_head, int d0, const void* q1,
                                   long long q1_token, long long q1_head, int d1, void* out, long long out_token,
                                   long long out_head, const void* keys, long long k_page, long long k_head, long long k_token,
@@ -122,8 +137,11 @@ LLM_EXPORT int llm_attention_rows(const void* q0, long long q0_token, long long 
                                   const int* page_table, int table_width, const int* token_request, const int* cu_tokens,
                                   const int* ctx_lens, const float* slopes, int n_tokens, int H, int KV, int page_size,
                                   int window, float scale, const float* sinks, const float* gate, long long gate_token,
-                                  int keep_first, int chunk, float softcap, cudaStream_t stream) {
+                                  int keep_first, int chunk, float softcap, int gate_per_head, int maps, long long q_map,
+                                  long long k_map, float diff_weight, float diff_eps, float diff_scale, const void* turn,
+                                  int turn_neighbours, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (maps < 1 || maps > 2 || (maps == 2 && (d1 != 0 || sinks)) || (turn && (dv & 1))) return LLM_ERR_BAD_ARGUMENT;
     if (keep_first < 0 || chunk < 0 || d0 <= 0 || d1 < 0 || d0 + d1 > MAX_DK || dv <= 0 || dv > MAX_DV || H <= 0 || KV <= 0 || H % KV || page_size <= 0 ||
         table_width <= 0 || (d1 > 0 && q1 == nullptr))
         return LLM_ERR_BAD_ARGUMENT;
@@ -141,7 +159,10 @@ LLM_EXPORT int llm_attention_rows(const void* q0, long long q0_token, long long 
         a.table_width = table_width; a.n_tokens = n_tokens; a.H = H; a.KV = KV; a.page_size = page_size; a.window = window;
         a.scale = scale; a.keep_first = keep_first; a.chunk = chunk; a.softcap = softcap;
         a.key_part = 0; a.keys1 = nullptr; a.k1_token = 0; a.fresh_d0 = 0; a.stats = nullptr;
-        a.sinks = sinks; a.gate = gate; a.gate_token = gate_token;
+        a.sinks = sinks; a.gate = gate; a.gate_token = gate_token; a.gate_per_head = gate_per_head;
+        a.maps = maps; a.q_map = q_map; a.k_map = k_map;
+        a.diff_weight = diff_weight; a.diff_eps = diff_eps; a.diff_scale = diff_scale;
+        a.turn = (const float2*)turn; a.turn_neighbours = turn_neighbours;
     };
     if (dtype == LLM_F32) {
         RowsArgs<float> a;
@@ -169,5 +190,5 @@ LLM_EXPORT int llm_attention_generic(const void* q, int q_stride, void* out, int
     const void* values = (const char*)pool + (size_t)KV * head * element;
     return llm_attention_rows(q, q_stride, D, D, nullptr, 0, 0, 0, out, out_stride, D, pool, page, head, D, values, page, head,
                               D, D, dtype, page_table, table_width, token_request, cu_tokens, ctx_lens, nullptr, n_tokens, H,
-                              KV, page_size, window, scale, nullptr, nullptr, 0, 0, 0, 0.f, stream);
+                              KV, page_size, window, scale, nullptr, nullptr, 0, 0, 0, 0.f, 0, 1, 0, 0, 0.f, 0.f, 0.f, nullptr, 0, stream);
 }

@@ -40,8 +40,44 @@ struct RowsArgs {
     // per query head (or null): one more term exp(sinks[h]) in the softmax's denominator, with no key and no value; it is
     // not scaled and counts once
     const float* sinks;
-    // [n_tokens, gate_token] float32 (or null): the output of head h, lane d is multiplied by sigmoid(gate[t, h * dv + d])
+    // [n_tokens, gate_token] float32 (or null): the output of head h, lane d is multiplied by sigmoid(gate[t, h * dv + d]),
+    // or, with gate_per_head, by sigmoid(gate[t, h])
     const float* gate;
     long long gate_token;
+    int gate_per_head;
+    // Two score maps a head over the same values (maps = 2; 1: an ordinary head).  A head's query of map m starts m * q_map
+    // elements behind its first lane, a key head's key of map m starts m * k_map behind its own, d0 lanes each (d1 = 0).
+    // Every map has a softmax of its own; with a1 and a2 their outputs the head's output is u / sqrt(mean(u^2) + diff_eps)
+    // * diff_scale over the head's dv lanes, u = a1 - diff_weight * a2.
+    int maps;
+    long long q_map, k_map;
+    float diff_weight, diff_eps, diff_scale;
+    // [n_tokens, dv / 2] (cos, sin) (or null): the values in the pages were turned by their own positions' angles; pair m of a
+    // head's output, lanes m and m + dv/2 (turn_neighbours: 2m and 2m + 1), is turned back by the query token's row
+    const float2* turn;
+    int turn_neighbours;
 };
+
+// The end of one head's output: y [dv] in shared memory, complete and visible to this warp; turned back where the values were
+// turned (`turn`: the token's row or null), gated (`gate`: the head's first gate or null, `gate_step` apart) and written.
+template <typename T>
+__device__ __forceinline__ void write_head(const float* y, int dv, int lane, const float2* turn, int neighbours, const float* gate,
+                                           int gate_step, T* out) {
+    auto put = [&](int d, float v) {
+        if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)d * gate_step]));
+        out[d] = from_float<T>(v);
+    };
+    if (turn) {
+        const int half = dv >> 1;
+        for (int m = lane; m < half; m += 32) {
+            const int a = neighbours ? 2 * m : m, b = neighbours ? 2 * m + 1 : m + half;
+            const float2 cs = turn[m];
+            const float u = y[a], v = y[b];
+            put(a, u * cs.x + v * cs.y);
+            put(b, v * cs.x - u * cs.y);
+        }
+    } else {
+        for (int d = lane; d < dv; d += 32) put(d, y[d]);
+    }
+}
 

@@ -10,6 +10,13 @@
 // Key tiles (64 keys, or 32 where rows are long) arrive by cp.async into a ring of two; keys past the request's length
 // are filled with zeros.  The keys of a row tile may be cut over `splits` CTAs, whose partial results (unnormalised
 // output, running maximum, sum) a second kernel merges.
+//
+// Heads of two score maps (MAPS = 2): a warp's sixteen rows are eight (token, group member) pairs, rows r and r + 8 the two maps
+// of one pair, so that a thread holds both maps' scores and outputs of its pair: keys and values cross shared memory once for
+// both maps, and the two outputs meet in registers.  A key row holds both maps' lanes; in the products of one map's lanes the
+// other map's rows are zeros.
+#include <type_traits>
+
 #include "attention_rows.cuh"
 
 namespace {
@@ -46,15 +53,16 @@ __device__ __forceinline__ unsigned pack2(float lo, float hi) {
 
 // BM rows a CTA (64 or 128: sixteen a warp).  The larger tile halves the trips of keys and values from L2 per row, which
 // is what bounds requests that bring many rows per key/value head.
-template <int DV_MAX, int BN, int BM>
+template <int DV_MAX, int BN, int BM, int MAPS>
 __global__ void __launch_bounds__(BM * 2, (DV_MAX <= 64 ? 4 : (DV_MAX <= 128 ? 3 : 2)) * 64 / BM)
 attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict__ part_o, float* __restrict__ part_ml) {
     constexpr int THREADS = BM * 2;
+    constexpr int TILE = BM / MAPS, WROWS = 16 / MAPS;  // (token, group member) pairs of the CTA and of a warp
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int dk = a.d0 + a.d1, dv = a.dv, kp = dk + PAD, vp = dv + PAD;
+    const int dk = MAPS * a.d0 + a.d1, dv = a.dv, kp = dk + PAD, vp = dv + PAD;
     const bool alias = a.key_part != 2 && a.values == a.keys && a.v_page == a.k_page && a.v_head == a.k_head && a.v_token == a.k_token;
-    bf16* Qs = reinterpret_cast<bf16*>(smem_raw);  // [BM][kp]
-    bf16* Ks = Qs + BM * kp;                       // [2][BN][kp]
+    bf16* Qs = reinterpret_cast<bf16*>(smem_raw);  // [TILE][kp]
+    bf16* Ks = Qs + TILE * kp;                       // [2][BN][kp]
     bf16* Vs = alias ? Ks : Ks + 2 * BN * kp;      // [2][BN][vp] unless the values are the head of the key rows
     const int v_pitch = alias ? kp : vp, v_stage = alias ? BN * kp : BN * vp;
 
@@ -64,13 +72,13 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
     const int tile = (int)(gridDim.x / splits) - 1 - slot;
     const int group = a.H / a.KV;
     const int q_begin = a.cu_tokens[r], q_len = a.cu_tokens[r + 1] - q_begin, ctx_len = a.ctx_lens[r];
-    const int rows_total = q_len * group, row0 = tile * BM;
+    const int rows_total = q_len * group, row0 = tile * TILE;
     if (row0 >= rows_total) return;
     const int first_pos = ctx_len - q_len;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
     // the keys this tile's rows see, and this split's share of their tiles
-    const int pos_min = first_pos + row0 / group, pos_max = first_pos + min(rows_total - 1, row0 + BM - 1) / group;
+    const int pos_min = first_pos + row0 / group, pos_max = first_pos + min(rows_total - 1, row0 + TILE - 1) / group;
     int key_lo = a.window > 0 ? max(0, pos_min - a.window + 1) : 0, key_hi = pos_max;
     if (a.chunk > 0) key_lo = max(key_lo, pos_min - pos_min % a.chunk);  // the oldest row's block of positions starts first
     if (a.key_part == 1) key_hi = min(key_hi, first_pos - 1);  // only what was cached before this step
@@ -132,13 +140,14 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
     };
 
     // queries of the tile's rows into shared memory (rows past the request's last are zeros)
-    for (int i = tid; i < BM * k_chunks; i += THREADS) {
+    for (int i = tid; i < TILE * k_chunks; i += THREADS) {
         const int row = i / k_chunks, c = (i - row * k_chunks) * 8, R = row0 + row;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (R < rows_total) {
             const int t = q_begin + R / group, h = kvh * group + R % group;
-            const bf16* src = c < a.d0 ? a.q0 + (long long)t * a.q0_token + (long long)h * a.q0_head + c
-                                       : a.q1 + (long long)t * a.q1_token + (long long)h * a.q1_head + (c - a.d0);
+            const bf16* src = MAPS == 2 ? a.q0 + (long long)t * a.q0_token + (long long)h * a.q0_head + (c < a.d0 ? c : a.q_map + (c - a.d0))
+                              : c < a.d0 ? a.q0 + (long long)t * a.q0_token + (long long)h * a.q0_head + c
+                                         : a.q1 + (long long)t * a.q1_token + (long long)h * a.q1_head + (c - a.d0);
             v = *reinterpret_cast<const uint4*>(src);
         }
         *reinterpret_cast<uint4*>(Qs + row * kp + c) = v;
@@ -146,12 +155,13 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
     if (t_begin < t_end) load_tile(t_begin, 0);
     cp_async_commit();
 
-    // the two rows of this thread: (lane / 4) and (lane / 4 + 8) of the warp's sixteen
+    // the two rows of this thread: (lane / 4) and (lane / 4 + 8) of the warp's sixteen (with two maps: one pair's)
+    auto pair_of = [&](int e) { return row0 + warp * WROWS + (lane >> 2) + (MAPS == 1 ? 8 * e : 0); };
     int pos[2], lo[2], hi[2];
     float slope[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-        const int R = min(row0 + warp * 16 + (lane >> 2) + 8 * e, rows_total - 1);
+        const int R = min(pair_of(e), rows_total - 1);
         pos[e] = first_pos + R / group;
         lo[e] = a.window > 0 ? max(0, pos[e] - a.window + 1) : 0;
         if (a.chunk > 0) lo[e] = max(lo[e], pos[e] - pos[e] % a.chunk);
@@ -163,7 +173,7 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
     // the keys that every row of this warp sees: from the newest row's window start to the oldest row's position
     int warp_lo, warp_hi;
     {
-        const int R0 = min(row0 + warp * 16, rows_total - 1), R1 = min(row0 + warp * 16 + 15, rows_total - 1);
+        const int R0 = min(row0 + warp * WROWS, rows_total - 1), R1 = min(row0 + warp * WROWS + WROWS - 1, rows_total - 1);
         const int p0 = first_pos + R0 / group, p1 = first_pos + R1 / group;
         warp_lo = a.window > 0 ? max(0, p1 - a.window + 1) : 0;
         if (a.chunk > 0) warp_lo = max(warp_lo, p1 - p1 % a.chunk);
@@ -176,7 +186,7 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
         // (a row's sum is kept in four lanes' shares until the end: the share of the first takes it)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-            const int R = min(row0 + warp * 16 + (lane >> 2) + 8 * e, rows_total - 1);
+            const int R = min(pair_of(e), rows_total - 1);
             m[e] = a.sinks[kvh * group + R % group] * LOG2E;
             l[e] = (lane & 3) == 0 ? 1.f : 0.f;
         }
@@ -201,7 +211,11 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
 #pragma unroll 2
         for (int ks = 0; ks < dk; ks += 16) {
             unsigned qa[4];
-            ldmatrix_x4(qa, Qs + (warp * 16 + (lane & 15)) * kp + ks + (lane >> 4) * 8);
+            ldmatrix_x4(qa, Qs + (warp * WROWS + (lane & (WROWS - 1))) * kp + ks + (lane >> 4) * 8);
+            if constexpr (MAPS == 2) {  // these lanes belong to one map: the rows of the other are zeros
+                if (ks < a.d0) qa[1] = qa[3] = 0u;
+                else qa[0] = qa[2] = 0u;
+            }
 #pragma unroll
             for (int nb = 0; nb < BN / 8; nb += 2) {
                 unsigned kb[4];
@@ -284,32 +298,13 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
         l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
     }
+    if (splits > 1) {
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-        const int R = row0 + warp * 16 + (lane >> 2) + 8 * e;
-        if (R >= rows_total) continue;
-        const int t = q_begin + R / group, h = kvh * group + R % group;
-        if (splits == 1) {
-            const float inv = l[e] > 0.f ? 1.f / l[e] : 0.f;  // no key seen (a part without keys for this row): zeros
-            if (a.stats && (lane & 3) == 0) {
-                a.stats[((size_t)t * a.H + h) * 2] = m[e];  // in units of log 2, as the merge expects
-                a.stats[((size_t)t * a.H + h) * 2 + 1] = l[e];
-            }
-            bf16* op = a.out + (long long)t * a.out_token + (long long)h * a.out_head;
-            const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (long long)h * dv : nullptr;
-#pragma unroll
-            for (int i = 0; i < DV_MAX / 8; ++i)
-                if (i * 8 < dv) {
-                    const int col = i * 8 + (lane & 3) * 2;
-                    float y0 = o[i][2 * e] * inv, y1 = o[i][2 * e + 1] * inv;
-                    if (gp) {
-                        y0 *= 1.f / (1.f + __expf(-gp[col]));
-                        y1 *= 1.f / (1.f + __expf(-gp[col + 1]));
-                    }
-                    *reinterpret_cast<__nv_bfloat162*>(op + col) = __floats2bfloat162_rn(y0, y1);
-                }
-        } else {
-            const size_t slot = ((size_t)t * a.H + h) * splits + split;
+        for (int e = 0; e < 2; ++e) {
+            const int R = pair_of(e);
+            if (R >= rows_total) continue;
+            const int t = q_begin + R / group, h = kvh * group + R % group;
+            const size_t slot = (((size_t)t * a.H + h) * MAPS + (MAPS == 2 ? e : 0)) * splits + split;
             float* po = part_o + slot * dv;
 #pragma unroll
             for (int i = 0; i < DV_MAX / 8; ++i)
@@ -322,49 +317,123 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
                 part_ml[slot * 2 + 1] = l[e];
             }
         }
+        return;
+    }
+    float inv[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) inv[e] = l[e] > 0.f ? 1.f / l[e] : 0.f;  // no key seen (a part without keys for this row): zeros
+    if constexpr (MAPS == 2) {  // the two maps meet: what follows reads the result as row e = 0
+        float ss = 0.f;
+        const float w1 = a.diff_weight * inv[1];
+#pragma unroll
+        for (int i = 0; i < DV_MAX / 8; ++i)
+            if (i * 8 < dv) {
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    o[i][c] = o[i][c] * inv[0] - w1 * o[i][2 + c];
+                    ss = fmaf(o[i][c], o[i][c], ss);
+                }
+            }
+        ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+        ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+        inv[0] = a.diff_scale / sqrtf(ss / (float)dv + a.diff_eps);
+    }
+    if (a.turn) {
+        // the pairs of lanes that turn together lie in other registers, or in other threads: a warp's rows go through shared memory
+        __syncthreads();  // the last tile has been read by all warps
+        float* stage = reinterpret_cast<float*>(smem_raw) + (size_t)warp * WROWS * dv;
+#pragma unroll
+        for (int e = 0; e < 3 - MAPS; ++e)
+#pragma unroll
+            for (int i = 0; i < DV_MAX / 8; ++i)
+                if (i * 8 < dv)
+                    *reinterpret_cast<float2*>(stage + ((lane >> 2) + 8 * e) * dv + i * 8 + (lane & 3) * 2) =
+                        make_float2(o[i][2 * e] * inv[e], o[i][2 * e + 1] * inv[e]);
+        __syncwarp();
+        for (int i = 0; i < WROWS; ++i) {
+            const int R = row0 + warp * WROWS + i;
+            if (R >= rows_total) break;
+            const int t = q_begin + R / group, h = kvh * group + R % group;
+            const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (a.gate_per_head ? (long long)h : (long long)h * dv) : nullptr;
+            write_head<bf16>(stage + i * dv, dv, lane, a.turn + (size_t)t * (dv >> 1), a.turn_neighbours, gp, a.gate_per_head ? 0 : 1,
+                             a.out + (long long)t * a.out_token + (long long)h * a.out_head);
+        }
+        return;
+    }
+#pragma unroll
+    for (int e = 0; e < 3 - MAPS; ++e) {
+        const int R = pair_of(e);
+        if (R >= rows_total) continue;
+        const int t = q_begin + R / group, h = kvh * group + R % group;
+        if (a.stats && (lane & 3) == 0) {
+            a.stats[((size_t)t * a.H + h) * 2] = m[e];  // in units of log 2, as the merge expects
+            a.stats[((size_t)t * a.H + h) * 2 + 1] = l[e];
+        }
+        bf16* op = a.out + (long long)t * a.out_token + (long long)h * a.out_head;
+        const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (a.gate_per_head ? (long long)h : (long long)h * dv) : nullptr;
+        const int gate_step = a.gate_per_head ? 0 : 1;
+#pragma unroll
+        for (int i = 0; i < DV_MAX / 8; ++i)
+            if (i * 8 < dv) {
+                const int col = i * 8 + (lane & 3) * 2;
+                float y0 = o[i][2 * e] * inv[e], y1 = o[i][2 * e + 1] * inv[e];
+                if (gp) {
+                    y0 *= 1.f / (1.f + __expf(-gp[col * gate_step]));
+                    y1 *= 1.f / (1.f + __expf(-gp[(col + 1) * gate_step]));
+                }
+                *reinterpret_cast<__nv_bfloat162*>(op + col) = __floats2bfloat162_rn(y0, y1);
+            }
     }
 }
 
-// out[t, h] = sum_s exp(m_s - M) o_s / sum_s exp(m_s - M) l_s over the splits' partial results; one warp per (token, head)
+// out[t, h] = sum_s exp(m_s - M) o_s / sum_s exp(m_s - M) l_s over the splits' partial results, for each of a head's maps; two
+// maps then meet, the result is turned back and gated, as in the kernel above.  One warp per (token, head); dv <= 256.
 __global__ void __launch_bounds__(128)
-attention_rows_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
-                            long long out_token, long long out_head, int n_tokens, int H, int dv, int splits,
-                            const float* __restrict__ gate, long long gate_token) {
-    const int lane = threadIdx.x & 31;
-    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+attention_rows_merge_kernel(const RowsArgs<bf16> a, const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits) {
+    __shared__ float rows_s[4][256];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dv = a.dv;
+    const long long item = (long long)blockIdx.x * 4 + warp;
     pdl_trigger();
     pdl_wait();
-    if (item >= (long long)n_tokens * H) return;
-    const int t = (int)(item / H), h = (int)(item - (long long)t * H);
-    const float* ml = part_ml + (size_t)item * splits * 2;
-    // lane s holds the weight of split s (at most 32 splits): exp(m_s - M), and the sum of all of them times their sums
-    const float ms = lane < splits ? ml[2 * lane] : -INFINITY, ls = lane < splits ? ml[2 * lane + 1] : 0.f;
-    const float M = warp_max(ms);
-    const float ws = ms == -INFINITY ? 0.f : exp2f(ms - M);  // the kernel's maxima are in units of log 2
-    const float inv = 1.f / warp_sum(ws * ls);
-    bf16* op = out + (long long)t * out_token + (long long)h * out_head;
-    const float* po = part_o + (size_t)item * splits * dv;
-    for (int d0 = 0; d0 < dv; d0 += 256) {  // eight independent sums a lane, so that a split's loads are in flight together
-        float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (item >= (long long)a.n_tokens * a.H) return;
+    const int t = (int)(item / a.H), h = (int)(item - (long long)t * a.H);
+    float y[8];
+    for (int map = 0; map < a.maps; ++map) {
+        const size_t first = ((size_t)item * a.maps + map) * splits;
+        const float* ml = part_ml + first * 2;
+        // lane s holds the weight of split s (at most 32 splits): exp(m_s - M), and the sum of all of them times their sums
+        const float ms = lane < splits ? ml[2 * lane] : -INFINITY, ls = lane < splits ? ml[2 * lane + 1] : 0.f;
+        const float M = warp_max(ms);
+        const float ws = ms == -INFINITY ? 0.f : exp2f(ms - M);  // the kernel's maxima are in units of log 2
+        const float inv = 1.f / warp_sum(ws * ls);
+        const float* po = part_o + first * dv;
+        float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};  // eight independent sums a lane: a split's loads are in flight together
         for (int s = 0; s < splits; ++s) {
             const float w = __shfl_sync(0xffffffffu, ws, s);
             if (w == 0.f) continue;  // uniform across the warp
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-                const int d = d0 + lane + 32 * i;
+                const int d = lane + 32 * i;
                 if (d < dv) acc[i] = fmaf(w, po[(size_t)s * dv + d], acc[i]);
             }
         }
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int d = d0 + lane + 32 * i;
-            if (d < dv) {
-                float y = acc[i] * inv;
-                if (gate) y *= 1.f / (1.f + __expf(-gate[(long long)t * gate_token + (long long)h * dv + d]));
-                op[d] = __float2bfloat16_rn(y);
-            }
-        }
+        for (int i = 0; i < 8; ++i) y[i] = map == 0 ? acc[i] * inv : y[i] - a.diff_weight * (acc[i] * inv);
     }
+    if (a.maps == 2) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ss = fmaf(y[i], y[i], ss);  // lanes beyond dv hold zeros
+        const float norm = a.diff_scale / sqrtf(warp_sum(ss) / (float)dv + a.diff_eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] *= norm;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) rows_s[warp][lane + 32 * i] = y[i];
+    __syncwarp();
+    const float* gp = a.gate ? a.gate + (long long)t * a.gate_token + (a.gate_per_head ? (long long)h : (long long)h * dv) : nullptr;
+    write_head<bf16>(rows_s[warp], dv, lane, a.turn ? a.turn + (size_t)t * (dv >> 1) : nullptr, a.turn_neighbours, gp,
+                     a.gate_per_head ? 0 : 1, a.out + (long long)t * a.out_token + (long long)h * a.out_head);
 }
 
 // out[t, h] = (w1 o1 + w2 o2) / (w1 + w2) with w = sum * 2^(maximum - M): two parts of one softmax, each normalised by
@@ -442,17 +511,17 @@ merge_project_gate_kernel(const float* __restrict__ part_o, const float* __restr
     }
 }
 
-template <int DV_MAX, int BN, int BM = 64>
+template <int DV_MAX, int BN, int BM = 64, int MAPS = 1>
 int launch(const RowsArgs<bf16>& a, int requests, int max_query_len, int splits, float* part_o, float* part_ml, size_t smem,
            cudaStream_t stream) {
     constexpr int THREADS = BM * 2;
-    auto kernel = attention_rows_mma_kernel<DV_MAX, BN, BM>;
+    auto kernel = attention_rows_mma_kernel<DV_MAX, BN, BM, MAPS>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
     const int group = a.H / a.KV;
-    const long long tiles = ((long long)max_query_len * group + BM - 1) / BM;
+    const long long tiles = ((long long)max_query_len * group + BM / MAPS - 1) / (BM / MAPS);
     if (tiles * splits > 0x7fffffffLL || a.KV > 65535 || requests > 65535) return LLM_ERR_UNSUPPORTED;
     return launch_pdl(kernel, dim3((unsigned)(tiles * splits), a.KV, requests), dim3(THREADS), smem, stream, a, splits, part_o, part_ml);
 }
@@ -461,7 +530,7 @@ int launch(const RowsArgs<bf16>& a, int requests, int max_query_len, int splits,
 
 // As llm_attention_rows, for bfloat16 with every run of lanes a multiple of 16 and 16-byte aligned rows; dv <= 256.
 // `max_query_len`: the most tokens a request brings (it sizes the grid).  `splits` > 1 cuts every row tile's keys over
-// that many CTAs; part_o [n_tokens * H * splits * dv] and part_ml [n_tokens * H * splits * 2] (float32) then hold the
+// that many CTAs; part_o [n_tokens * H * maps * splits * dv] and part_ml [n_tokens * H * maps * splits * 2] (float32) then hold the
 // partial results until the merge that follows.  Returns LLM_ERR_UNSUPPORTED for shapes it does not take.
 LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long long q0_head, int d0, const void* q1,
                                       long long q1_token, long long q1_head, int d1, void* out, long long out_token,
@@ -472,12 +541,17 @@ LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long l
                                       int n_tokens, int requests, int max_query_len, int H, int KV, int page_size, int window,
                                       float scale, int splits, float* part_o, float* part_ml, int key_part, const void* keys1,
                                       long long k1_token, int fresh_d0, float* stats, const float* sinks, const float* gate,
-                                      long long gate_token, int keep_first, int chunk, float softcap, cudaStream_t stream) {
+                                      long long gate_token, int keep_first, int chunk, float softcap, int gate_per_head, int maps,
+                                      long long q_map, long long k_map, float diff_weight, float diff_eps, float diff_scale,
+                                      const void* turn, int turn_neighbours, cudaStream_t stream) {
     if (n_tokens <= 0 || requests <= 0) return 0;
+    if (maps < 1 || maps > 2 || (maps == 2 && (d1 != 0 || sinks || key_part != 0 || stats)) || (turn && (key_part != 0 || stats)))
+        return LLM_ERR_BAD_ARGUMENT;
+    if (maps == 2 && (k_map != d0 || (q_map & 7))) return LLM_ERR_UNSUPPORTED;
     if (d0 <= 0 || d1 < 0 || dv <= 0 || H <= 0 || KV <= 0 || H % KV || page_size <= 0 || table_width <= 0 || splits < 1 ||
         max_query_len < 1 || (d1 > 0 && q1 == nullptr) || (splits > 1 && (part_o == nullptr || part_ml == nullptr)))
         return LLM_ERR_BAD_ARGUMENT;
-    const int dk = d0 + d1;
+    const int dk = maps * d0 + d1;
     auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
     if ((d0 & 15) || (d1 & 15) || (dv & 15) || dv > 256 || dk > 640) return LLM_ERR_UNSUPPORTED;
     if (key_part < 0 || key_part > 2 || (stats && splits != 1)) return LLM_ERR_BAD_ARGUMENT;
@@ -504,32 +578,43 @@ LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long l
     a.scale = scale; a.keep_first = keep_first; a.chunk = chunk; a.softcap = softcap;
     a.key_part = key_part; a.keys1 = key_part == 2 ? (const bf16*)keys1 : nullptr; a.k1_token = k1_token; a.fresh_d0 = fresh_d0;
     a.stats = stats;
-    a.sinks = sinks; a.gate = gate; a.gate_token = gate_token;
+    a.sinks = sinks; a.gate = gate; a.gate_token = gate_token; a.gate_per_head = gate_per_head;
+    a.maps = maps; a.q_map = q_map; a.k_map = k_map;
+    a.diff_weight = diff_weight; a.diff_eps = diff_eps; a.diff_scale = diff_scale;
+    a.turn = (const float2*)turn; a.turn_neighbours = turn_neighbours;
     const bool alias = key_part != 2 && values == keys && v_page == k_page && v_head == k_head && v_token == k_token;
-    auto smem_for = [&](int bn, int bm = 64) { return (size_t)(bm + 2 * bn) * (dk + PAD) * 2 + (alias ? 0 : (size_t)2 * bn * (dv + PAD) * 2); };
+    // a tile's queries, two stages of keys and of values; at the end, where values turn back, the tile's rows in 32-bit instead
+    auto smem_for = [&](int bn, int bm = 64) {
+        const size_t ring = (size_t)(bm / maps + 2 * bn) * (dk + PAD) * 2 + (alias ? 0 : (size_t)2 * bn * (dv + PAD) * 2);
+        const size_t stage = turn ? (size_t)(bm / maps) * dv * 4 : 0;
+        return ring > stage ? ring : stage;
+    };
     const bool wide = smem_for(64) <= 160 * 1024;
     size_t smem = smem_for(wide ? 64 : 32);
     if (smem > 220 * 1024) return LLM_ERR_UNSUPPORTED;
     int code;
     // many rows per key/value head (long prompt portions), values of at most 128 lanes: 128 rows a CTA
-    const bool tall = wide && dv <= 128 && (long long)max_query_len * (H / KV) >= 512 && smem_for(64, 128) <= 100 * 1024;
-    if (tall) {
-        smem = smem_for(64, 128);
-        code = dv <= 64 ? launch<64, 64, 128>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
-                        : launch<128, 64, 128>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
-    } else if (dv <= 64)
-        code = wide ? launch<64, 64>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
-                    : launch<64, 32>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
-    else if (dv <= 128)
-        code = wide ? launch<128, 64>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
-                    : launch<128, 32>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
-    else
-        code = wide ? launch<256, 64>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
-                    : launch<256, 32>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
+    const bool tall = wide && dv <= 128 && (long long)max_query_len * (H / KV) * maps >= 512 && smem_for(64, 128) <= 100 * 1024;
+    if (tall) smem = smem_for(64, 128);
+    auto go = [&](auto maps_tag) {
+        constexpr int MAPS = decltype(maps_tag)::value;
+        if (tall)
+            return dv <= 64 ? launch<64, 64, 128, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
+                            : launch<128, 64, 128, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
+        if (dv <= 64)
+            return wide ? launch<64, 64, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
+                        : launch<64, 32, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
+        if (dv <= 128)
+            return wide ? launch<128, 64, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
+                        : launch<128, 32, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
+        return wide ? launch<256, 64, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream)
+                    : launch<256, 32, 64, MAPS>(a, requests, max_query_len, splits, part_o, part_ml, smem, stream);
+    };
+    code = maps == 2 ? go(std::integral_constant<int, 2>{}) : go(std::integral_constant<int, 1>{});
     if (code != 0 || splits == 1 || out == nullptr) return code;  // no out: the partial results are what the caller wants
     const long long items = (long long)n_tokens * H;
-    return launch_pdl(attention_rows_merge_kernel, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, (const float*)part_o,
-                      (const float*)part_ml, (bf16*)out, out_token, out_head, n_tokens, H, dv, splits, gate, gate_token);
+    return launch_pdl(attention_rows_merge_kernel, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, a, (const float*)part_o,
+                      (const float*)part_ml, splits);
 }
 
 // The partial results of llm_attention_rows_mma with splits > 1 and no out (part_o, part_ml), merged, multiplied per head

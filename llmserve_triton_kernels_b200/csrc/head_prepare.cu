@@ -4,14 +4,18 @@
 // values_are_keys: no value columns, a key head's value is that head as projected, bias included, before norm and
 // rotation).  In this order, each step optional:
 //   bias:      the stacked bias (float32, laid out like the row) is added
-//   norm:      every query head and every key head is divided by sqrt(mean(x^2) + eps) over its D lanes and multiplied
-//              by qw / kw [D], the same for every head
+//   norm:      1: every query head and every key head is divided by sqrt(mean(x^2) + eps) over its D lanes and multiplied
+//              by qw / kw [D], the same for every head; 2: all query heads together are, over their Hq * D lanes, by
+//              qw [Hq * D], all key heads likewise by kw [Hk * D]
 //   rotate:    lanes i and i + rot/2 (i < rot/2) of every head turn by position * freq[i]; lanes >= rot pass
 //              (interleaved: lanes 2i and 2i + 1 instead)
+//   turn:      with v_freq [V / 2] every value head's pairs (lanes m and m + V/2, or 2m and 2m + 1) turn by
+//              position * v_freq[m]; turn_out [N, V / 2] takes the (cos, sin) for whoever turns them back
 //   values:    v_keep [N, Hk * V] (float32) takes the values as projected, bias included; or, with v_first [N, Hk * V],
 //              the values become (1 - v_lambda) v + v_lambda v_first (those of the same token in an earlier layer)
 //   warm:      queries times 1 + coef * ln(floor((position + 1) / every) + 1)
-// Queries go to q_out [N, Hq * D]; keys and values into the token's slot of pool [pages, 2, Hk, page_size, Dp].
+// Queries go to q_out [N, Hq * D]; keys and values into the token's slot of pool [pages, 2, Hk, page_size, Dp].  With maps = 2
+// every two key heads in a row share a value head and a row of the pool [pages, 2, Hk / 2, page_size, Dp], side by side.
 // Everything is computed in 32-bit.  One CTA per token, one warp per head at a time.
 #include <type_traits>
 
@@ -28,30 +32,54 @@ head_prepare_kernel(const TI* __restrict__ proj, int ldp, const float* __restric
                     const float* __restrict__ kw, float eps, int normed, const float* __restrict__ freq, int rot,
                     const int* __restrict__ positions, float warm_coef, int warm_every, int Hq, int Hk, int D, int V,
                     int values_are_keys, int interleaved, float* __restrict__ v_keep, const float* __restrict__ v_first,
-                    float v_lambda) {
-    extern __shared__ float smem[];  // [WARPS][D] a head as projected, then rot/2 (cos, sin) pairs
+                    float v_lambda, int maps, const float* __restrict__ v_freq, float2* __restrict__ turn_out) {
+    extern __shared__ float smem[];  // [WARPS][D] a head as projected, then rot/2 (cos, sin) pairs, then V/2 for the values
+    __shared__ float scratch[33];
     float2* turn = reinterpret_cast<float2*>(smem + WARPS * D + ((WARPS * D) & 1));
     pdl_trigger();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int half = rot >> 1;
-    const int position = (half > 0 || warm_every > 0) ? positions[t] : 0;
+    const int position = (half > 0 || warm_every > 0 || v_freq) ? positions[t] : 0;
+    float2* v_turn = turn + half;
+    const int v_half = v_freq ? V >> 1 : 0, Gv = Hk / maps;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
         sincosf((float)position * freq[i], &s, &c);
         turn[i] = make_float2(c, s);
+    }
+    for (int i = threadIdx.x; i < v_half; i += blockDim.x) {
+        float s, c;
+        sincosf((float)position * v_freq[i], &s, &c);
+        v_turn[i] = make_float2(c, s);
     }
     const float warm = warm_every > 0 ? 1.f + warm_coef * logf((float)((position + 1) / warm_every) + 1.f) : 1.f;
     const int slot = Hk > 0 ? slot_map[t] : 0;
     const int page = slot / page_size, off = slot % page_size;
     __syncthreads();
     pdl_wait();
+    if (turn_out)
+        for (int i = threadIdx.x; i < v_half; i += blockDim.x) turn_out[(size_t)t * v_half + i] = v_turn[i];
     const TI* row = proj + (size_t)t * ldp;
+    float whole[2] = {1.f, 1.f};  // the scales of all query heads and of all key heads together
+    if (normed == 2) {
+        float sums[2] = {0.f, 0.f};
+        for (int i = threadIdx.x; i < (Hq + Hk) * D; i += blockDim.x) {
+            float v = to_float(row[i]);
+            if (bias) v += bias[i];
+            if (i < Hq * D) sums[0] = fmaf(v, v, sums[0]);
+            else sums[1] = fmaf(v, v, sums[1]);
+        }
+        for (int e = 0; e < 2; ++e) {
+            const float ss = block_sum(sums[e], scratch);
+            whole[e] = 1.f / sqrtf(ss / (float)((e ? Hk : Hq) * D) + eps);
+        }
+    }
     float* buf = smem + warp * D;
     const int per_head = D - half;  // work items a head: `half` pairs, then the lanes that pass
     for (int head = warp; head < Hq + Hk; head += WARPS) {
         const bool is_q = head < Hq;
         const int base = head * D;  // keys follow the queries in the row and in the bias
-        TK* vdst = (!is_q && values_are_keys) ? pool + ((((size_t)page * 2 + 1) * Hk + (head - Hq)) * page_size + off) * Dp : nullptr;
+        TK* vdst = (!is_q && values_are_keys) ? pool + ((((size_t)page * 2 + 1) * Hk + (head - Hq)) * page_size + off) * Dp : nullptr;  // (one map)
         float ss = 0.f;
         for (int d = lane; d < D; d += 32) {
             float v = to_float(row[base + d]);
@@ -61,8 +89,9 @@ head_prepare_kernel(const TI* __restrict__ proj, int ldp, const float* __restric
             if (vdst) vdst[d] = from_float<TK>(v);
         }
         ss = warp_sum(ss);
-        const float ns = normed ? 1.f / sqrtf(ss / (float)D + eps) : 1.f;
+        const float ns = normed == 1 ? 1.f / sqrtf(ss / (float)D + eps) : normed == 2 ? whole[is_q ? 0 : 1] : 1.f;
         const float* w = normed ? (is_q ? qw : kw) : nullptr;
+        if (normed == 2) w += (is_q ? head : head - Hq) * D;
         const float post = is_q ? warm : 1.f;
         __syncwarp();
         for (int i = lane; i < per_head; i += 32) {
@@ -86,7 +115,8 @@ head_prepare_kernel(const TI* __restrict__ proj, int ldp, const float* __restric
                 dst[da] = from_float<TQ>(a);
                 if (db >= 0) dst[db] = from_float<TQ>(b);
             } else {
-                TK* dst = pool + (((size_t)page * 2 * Hk + (head - Hq)) * page_size + off) * Dp;
+                const int kh = (head - Hq) / maps;
+                TK* dst = pool + (((size_t)page * 2 * Gv + kh) * page_size + off) * Dp + (head - Hq - kh * maps) * D;
                 dst[da] = from_float<TK>(a);
                 if (db >= 0) dst[db] = from_float<TK>(b);
             }
@@ -95,13 +125,26 @@ head_prepare_kernel(const TI* __restrict__ proj, int ldp, const float* __restric
     }
     if (Hk > 0 && !values_are_keys) {
         const int vbase = (Hq + Hk) * D;
-        for (int i = threadIdx.x; i < Hk * V; i += blockDim.x) {
+        if (v_freq) {
+            for (int i = threadIdx.x; i < Gv * v_half; i += blockDim.x) {
+                const int kh = i / v_half, m = i - kh * v_half;
+                const int da = interleaved ? 2 * m : m, db = interleaved ? 2 * m + 1 : m + v_half;
+                float u = to_float(row[vbase + kh * V + da]), v = to_float(row[vbase + kh * V + db]);
+                if (bias) { u += bias[vbase + kh * V + da]; v += bias[vbase + kh * V + db]; }
+                const float2 cs = v_turn[m];
+                TK* dst = pool + ((((size_t)page * 2 + 1) * Gv + kh) * page_size + off) * Dp;
+                dst[da] = from_float<TK>(u * cs.x - v * cs.y);
+                dst[db] = from_float<TK>(v * cs.x + u * cs.y);
+            }
+            return;
+        }
+        for (int i = threadIdx.x; i < Gv * V; i += blockDim.x) {
             const int kh = i / V, d = i % V;
             float v = to_float(row[vbase + i]);
             if (bias) v += bias[vbase + i];
-            if (v_keep) v_keep[(size_t)t * Hk * V + i] = v;
-            if (v_first) v = (1.f - v_lambda) * v + v_lambda * v_first[(size_t)t * Hk * V + i];
-            pool[((((size_t)page * 2 + 1) * Hk + kh) * page_size + off) * Dp + d] = from_float<TK>(v);
+            if (v_keep) v_keep[(size_t)t * Gv * V + i] = v;
+            if (v_first) v = (1.f - v_lambda) * v + v_lambda * v_first[(size_t)t * Gv * V + i];
+            pool[((((size_t)page * 2 + 1) * Gv + kh) * page_size + off) * Dp + d] = from_float<TK>(v);
         }
     }
 }
@@ -113,18 +156,22 @@ LLM_EXPORT int llm_head_prepare(const void* proj, int in_dtype, int ldp, const f
                                 int out_dtype, const int* slot_map, int page_size, int Dp, const float* qw, const float* kw, float eps,
                                 int normed, const float* freq, int rot, const int* positions, float warm_coef, int warm_every, int N,
                                 int Hq, int Hk, int D, int V, int values_are_keys, int interleaved, float* v_keep,
-                                const float* v_first, float v_lambda, cudaStream_t stream) {
+                                const float* v_first, float v_lambda, int maps, const float* v_freq, void* turn_out, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (rot < 0 || rot % 2 || rot > D || Hq < 0 || Hk < 0 || D <= 0 || D > 1024 || (Hk > 0 && (!pool || !slot_map || Dp < D || page_size <= 0)) ||
+    if (maps < 1 || Hk % maps || (maps > 1 && values_are_keys) || normed < 0 || normed > 2 ||
+        (v_freq && (V & 1 || values_are_keys || Hk <= 0 || v_keep || v_first || !positions)) || (turn_out && !v_freq))
+        return LLM_ERR_BAD_ARGUMENT;
+    if (rot < 0 || rot % 2 || rot > D || Hq < 0 || Hk < 0 || D <= 0 || D > 1024 || (Hk > 0 && (!pool || !slot_map || Dp < maps * D || page_size <= 0)) ||
         (Hk > 0 && !values_are_keys && (V <= 0 || Dp < V)) || ((rot > 0 || warm_every > 0) && !positions) || (rot > 0 && !freq) ||
         (normed && (!qw || (Hk > 0 && !kw))) || (Hq > 0 && !q_out) || ((v_keep || v_first) && (values_are_keys || Hk <= 0)))
         return LLM_ERR_BAD_ARGUMENT;
     using bf = __nv_bfloat16;
-    const size_t smem = ((size_t)WARPS * D + 1) * sizeof(float) + (size_t)(rot / 2 + 1) * sizeof(float2);
+    const size_t smem = ((size_t)WARPS * D + 1) * sizeof(float) + (size_t)(rot / 2 + 1 + (v_freq ? V / 2 : 0)) * sizeof(float2);
     auto go = [&](auto kernel, auto* in, auto* qo) {
         using TK = std::remove_pointer_t<decltype(qo)>;
         return launch_pdl(kernel, dim3(N), dim3(WARPS * 32), smem, stream, in, ldp, bias, qo, ldq, (TK*)pool, slot_map, page_size, Dp, qw, kw,
-                          eps, normed, freq, rot, positions, warm_coef, warm_every, Hq, Hk, D, V, values_are_keys, interleaved, v_keep, v_first, v_lambda);
+                          eps, normed, freq, rot, positions, warm_coef, warm_every, Hq, Hk, D, V, values_are_keys, interleaved, v_keep, v_first, v_lambda, maps, v_freq,
+                          (float2*)turn_out);
     };
     if (in_dtype == LLM_F32 && out_dtype == LLM_F32) return go(head_prepare_kernel<float, float, float>, (const float*)proj, (float*)q_out);
     if (in_dtype == LLM_F32 && out_dtype == LLM_BF16) return go(head_prepare_kernel<float, bf, bf>, (const float*)proj, (bf*)q_out);

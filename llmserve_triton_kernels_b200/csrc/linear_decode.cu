@@ -299,7 +299,7 @@ LLM_EXPORT int llm_linear_decode_parts(int N) { return (N + 15) / 16; }
 //   mode 1: w = [gate | up] with the up rows starting at row up_offset; out [M, N] = silu(gate) * up.
 //   mode 2: resid [M, N] += product; xw_out [M, N] = resid * norm_w; ss_out [parts(N), M] = partial sums
 //           of resid^2.  out is not used.
-//   mode 4: mode 0 with the square of relu on the product.
+//   mode 4: mode 0 with the square of relu on the product; mode 6: with gelu (erf form).
 //   mode 5: resid [M, N] += resid_scale * product and nothing else (norm_w, xw_out, ss_out are not used).
 // in_ss (or null): [in_parts, M] partial sums of squares; the product is scaled by
 // rsqrt(sum / K + in_eps) per row.  Needs M <= 16, K a multiple of 64 (the weights travel in pieces of 64 k), 16-byte aligned rows;
@@ -338,8 +338,8 @@ LLM_EXPORT int llm_linear_decode(const void* x, const void* w, void* out, int ou
         p.resid_scale = resid_scale;
         return dispatch<MODE_RESIDUAL, __nv_bfloat16>(p, stream);
     }
-    if (mode == 4) {
-        p.act = 1;
+    if (mode == 4 || mode == 6) {
+        p.act = mode == 4 ? 1 : 2;
         mode = MODE_PLAIN;
     }
     if (mode == MODE_RESIDUAL) {

@@ -46,7 +46,7 @@ struct LinearParams {
     __nv_bfloat16* xw_out;  // MODE_RESIDUAL: [M, N] = resid * norm_w
     float* ss_out;          // MODE_RESIDUAL: [tiles of 16 features, M]
     float resid_scale;      // MODE_RESIDUAL: the product enters the stream times this
-    int act;                // MODE_PLAIN: 0 the product as it is, 1 the square of its relu
+    int act;                // MODE_PLAIN: 0 the product as it is, 1 the square of its relu, 2 its gelu (erf form)
     int* error_flag;        // set to 1 if a wait for a copy gave up (host-visible memory), or null
     int group;              // warps that share a tile: 1, 2, 4 or 8
     int slots;              // boxes of a warp's ring: 2 to SLOTS
@@ -454,6 +454,8 @@ __device__ __forceinline__ bool stream_run(StreamState& st, const LinearParams& 
                         if (p.act == 1) {
                             r = fmaxf(r, 0.f);
                             r *= r;
+                        } else if (p.act == 2) {
+                            r = 0.5f * r * (1.f + erff(r * 0.7071067811865476f));
                         }
                         reinterpret_cast<TO*>(p.out)[(size_t)m * p.ldo + n] = from_float<TO>(r);
                     }

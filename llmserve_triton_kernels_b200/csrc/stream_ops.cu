@@ -174,13 +174,14 @@ __global__ void stream_inject_kernel(float* __restrict__ resid, const TD* __rest
 }
 
 // ---------------------------------------------------------------------------------------------
-// one-input functions of a matrix with a row pitch: 0 relu(v)^2, 1 gelu (tanh form), 2 alpha * v, 3 silu
+// one-input functions of a matrix with a row pitch: 0 relu(v)^2, 1 gelu (tanh form), 2 alpha * v, 3 silu, 4 gelu (erf form)
 // ---------------------------------------------------------------------------------------------
 __device__ __forceinline__ float unary_of(float v, int kind, float alpha) {
     switch (kind) {
         case 0: v = fmaxf(v, 0.f); return v * v;
         case 1: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
         case 2: return alpha * v;
+        case 4: return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
         default: return v * sigmoid_f(v);
     }
 }
@@ -300,7 +301,7 @@ LLM_EXPORT int llm_stream_inject(float* resid, const void* delta, int delta_dtyp
 LLM_EXPORT int llm_unary(const void* x, int ldx, void* out, int ldo, int dtype, int rows, int cols, int kind, float alpha,
                          cudaStream_t stream) {
     if (rows <= 0 || cols <= 0) return 0;
-    if (ldx < cols || ldo < cols || kind < 0 || kind > 3) return LLM_ERR_BAD_ARGUMENT;
+    if (ldx < cols || ldo < cols || kind < 0 || kind > 4) return LLM_ERR_BAD_ARGUMENT;
     const size_t total = (size_t)rows * cols;
     const bool wide = ((cols | ldx | ldo) & 3) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0;
     const int threads = 256, blocks = flat_blocks(wide ? (total + 3) / 4 : total, threads);

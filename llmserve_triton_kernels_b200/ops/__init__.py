@@ -52,9 +52,11 @@ _SIGNATURES = {
     "llm_merge_two_parts": [_vp, _ll, _ll, _vp, _vp, _ll, _ll, _vp, _vp, _ll, _ll, _i, _i, _i, _vp],
     "llm_unit_norm_kv_write": [_vp, _i, _i, _vp, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "llm_attention_rows": [_vp, _ll, _ll, _i, _vp, _ll, _ll, _i, _vp, _ll, _ll, _vp, _ll, _ll, _ll, _vp, _ll, _ll, _ll, _i, _i,
-                           _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _ll, _i, _i, _f, _vp],
+                           _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _ll, _i, _i, _f,
+                           _i, _i, _ll, _ll, _f, _f, _f, _vp, _i, _vp],
     "llm_attention_rows_mma": [_vp, _ll, _ll, _i, _vp, _ll, _ll, _i, _vp, _ll, _ll, _vp, _ll, _ll, _ll, _vp, _ll, _ll, _ll, _i,
-                               _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp, _ll, _i, _vp, _vp, _vp, _ll, _i, _i, _f, _vp],
+                               _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp, _ll, _i, _vp, _vp, _vp, _ll, _i, _i, _f,
+                               _i, _i, _ll, _ll, _f, _f, _f, _vp, _i, _vp],
     "llm_gemm_simt_batched": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _ll, _ll, _ll, _vp],
     "llm_sample": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
     "llm_sigmoid_attention": [_vp, _i, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i,
@@ -66,7 +68,8 @@ _SIGNATURES = {
     "llm_head_norm_gate": [_vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _f, _i, _vp, _vp],
     "llm_embed_copies": [_vp, _vp, _i, _vp, _i, _i, _i, _i, _vp],
     "llm_hyper_mix_norm": [_vp, _vp, _vp, _vp, _vp, _f, _f, _f, _f, _i, _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp],
-    "llm_head_prepare": [_vp, _i, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _f, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp],
+    "llm_head_prepare": [_vp, _i, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _f, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _i, _vp, _vp, _vp],
+    "llm_shift_norm": [_vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "llm_short_conv": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "llm_row_rmsnorm": [_vp, _i, _i, _vp, _f, _vp, _i, _i, _i, _i, _vp],
     "llm_gated_scan": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _f, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
@@ -479,16 +482,18 @@ class ResidualSink:
         return NormedInput(xw, ss, self.eps, self.norm)
 
 
-def _decode_linear(x, w, out_dtype, mode: int, n_out: int, up_offset: int = 0):
-    """The weight-streaming product for few rows; None if it refuses the shape."""
+def _decode_linear(x, w, out_dtype, mode: int, n_out: int, up_offset: int = 0, out: torch.Tensor | None = None):
+    """The weight-streaming product for few rows (into ``out``, whose rows may have a pitch, if it is given); None if it
+    refuses the shape."""
     scaled = isinstance(x, NormedInput)
     xt = x.xw if scaled else x
     m, k = xt.shape
     if not (xt.dtype == torch.bfloat16 and m <= _DECODE_LINEAR_MAX_ROWS and xt.stride(1) == 1 and w.is_contiguous()):
         return None
-    out = torch.empty((m, n_out), dtype=out_dtype, device=xt.device)
+    if out is None:
+        out = torch.empty((m, n_out), dtype=out_dtype, device=xt.device)
     code = _launch(
-        "llm_linear_decode", _ptr(xt), _ptr(w), _ptr(out), _code(out_dtype), m, n_out, k, xt.stride(0), n_out,
+        "llm_linear_decode", _ptr(xt), _ptr(w), _ptr(out), _code(out_dtype), m, n_out, k, xt.stride(0), out.stride(0),
         _ptr(x.ss) if scaled else None, x.ss.shape[0] if scaled else 0, x.eps if scaled else 0.0, mode, up_offset,
         None, None, None, None, 1.0, _error_flag_ptr(), _stream(),
     )
@@ -879,7 +884,7 @@ def sample(
 # ------------------------------------------------------------------------------------------------
 # Operations of layers that normalise in groups, scale their contributions, gate their outputs, keep a recurrent
 # state, or attend over a latent (csrc/stream_ops.cu, recurrent.cu, cache_write.cu, attention_generic.cu).
-_UNARY_KINDS = {"relu2": 0, "gelu_tanh": 1, "scale": 2, "silu": 3}
+_UNARY_KINDS = {"relu2": 0, "gelu_tanh": 1, "scale": 2, "silu": 3, "gelu": 4}
 _GATE_KINDS = {"sigmoid": 0, "silu": 1}
 
 
@@ -940,27 +945,59 @@ def stream_inject(
     _check(code, "stream_inject")
 
 
-def unary(x: torch.Tensor, kind: str, alpha: float = 1.0, inplace: bool = False) -> torch.Tensor:
-    """A one-input function of every element, computed in 32-bit: ``relu2`` (the square of relu), ``gelu_tanh``,
-    ``silu``, or ``scale`` (``alpha * x``).  ``x [N, C]`` may have a row pitch."""
+def unary(x: torch.Tensor, kind: str, alpha: float = 1.0, inplace: bool = False, out: torch.Tensor | None = None) -> torch.Tensor:
+    """A one-input function of every element, computed in 32-bit: ``relu2`` (the square of relu), ``gelu_tanh``, ``gelu``
+    (the erf form), ``silu``, or ``scale`` (``alpha * x``).  ``x [N, C]`` and ``out`` may have a row pitch."""
     _need(kind in _UNARY_KINDS, f"no one-input function {kind!r}; known: {sorted(_UNARY_KINDS)}")
     _need(x.dim() == 2 and x.stride(1) == 1, "unary: a matrix with unit inner stride")
-    out = x if inplace else torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    if out is None:
+        out = x if inplace else torch.empty(x.shape, dtype=x.dtype, device=x.device)
+    _need(out.shape == x.shape and out.dtype == x.dtype and out.stride(1) == 1, "unary: the result has the input's shape and type")
     code = _launch("llm_unary", _ptr(x), x.stride(0), _ptr(out), out.stride(0), _code(x.dtype), x.shape[0], x.shape[1],
                    _UNARY_KINDS[kind], float(alpha), _stream())
     _check(code, "unary")
     return out
 
 
-def linear_act(x, w: torch.Tensor, activation: str) -> torch.Tensor:
+_DECODE_ACT_MODES = {"relu2": 4, "gelu": 6}  # activations that the weight-streaming product can end with
+
+
+def linear_act(x, w: torch.Tensor, activation: str, out: torch.Tensor | None = None) -> torch.Tensor:
     """``act(x @ w^T)`` for a one-input activation (see :func:`unary`): the product, then the activation on its
-    result in place; for few bfloat16 rows the square of relu is the end of the weight-streaming product itself."""
+    result in place; for few bfloat16 rows the square of relu and gelu (erf form) are the end of the weight-streaming product
+    itself.  ``out``: where the result goes (rows may have a pitch)."""
     xt = x.xw if isinstance(x, NormedInput) else x
-    if activation == "relu2" and xt.dtype == torch.bfloat16 and xt.shape[0] <= _DECODE_LINEAR_MAX_ROWS:
-        out = _decode_linear(x, w, torch.bfloat16, 4, w.shape[0])
-        if out is not None:
-            return out
-    return unary(linear(x, w), activation, inplace=True)
+    _need(out is None or (tuple(out.shape) == (xt.shape[0], w.shape[0]) and out.dtype == xt.dtype and out.stride(1) == 1), "linear_act: out [M, N] of the input's type")
+    if activation in _DECODE_ACT_MODES and xt.dtype == torch.bfloat16 and xt.shape[0] <= _DECODE_LINEAR_MAX_ROWS:
+        done = _decode_linear(x, w, torch.bfloat16, _DECODE_ACT_MODES[activation], w.shape[0], out=out)
+        if done is not None:
+            return done
+    return unary(linear(x, w), activation, inplace=out is None, out=out)
+
+
+def shift_norm(x: torch.Tensor, w1: torch.Tensor, eps: float, w2: torch.Tensor | None = None, shift: torch.Tensor | None = None,
+               states: torch.Tensor | None = None, ctx=None, state_slots: torch.Tensor | None = None,
+               out_dtype: torch.dtype = torch.float32) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """Two RMS norms of the same rows ``x [N, W]`` (float32): ``h = x * rsqrt(mean(x^2) + eps) * w1`` and, with ``w2``, the same
+    times ``w2``.  With ``shift`` (float32 ``[W]``) the first is ``h_t + shift * (h_(t-1) - h_t)``: ``h_(t-1)`` belongs to the
+    token in front in the same request (``ctx.token_request``, ``ctx.cu_tokens``), for a request's first row of the step it is
+    read from ``states[state_slots[r]]`` (float32 ``[slots, W]``, zeros at a request's start), which is then moved on to ``h``
+    of the request's last row.  Returns ``(shifted, second or None)`` in ``out_dtype``."""
+    _need(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), "shift_norm: the rows are contiguous float32 [N, W]")
+    n, w = x.shape
+    for t in (w1, w2, shift):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == w), "shift_norm: weights and shift are float32 [W]")
+    if shift is not None:
+        _need(states is not None and states.dtype == torch.float32 and states.is_contiguous() and tuple(states.shape[1:]) == (w,), "shift_norm: states [slots, W] float32")
+        _i32(state_slots, "state_slots")
+    first = torch.empty((n, w), dtype=out_dtype, device=x.device)
+    second = torch.empty((n, w), dtype=out_dtype, device=x.device) if w2 is not None else None
+    shifted = shift is not None
+    code = _launch("llm_shift_norm", _ptr(x), _ptr(w1), _ptr(w2), _ptr(shift), float(eps), _ptr(states) if shifted else None,
+                   _ptr(state_slots) if shifted else None, _ptr(ctx.token_request) if shifted else None, _ptr(ctx.cu_tokens) if shifted else None,
+                   _ptr(first), _ptr(second), _code(out_dtype), n, w, _stream())
+    _check(code, "shift_norm")
+    return first, second
 
 
 def gate_mul(a: torch.Tensor, b: torch.Tensor, kind: str = "sigmoid", per_head: bool = False) -> torch.Tensor:
@@ -1065,7 +1102,9 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
                    num_kv_heads: int, scale: float, window: int | None = None, slopes: torch.Tensor | None = None,
                    key_part: int = 0, keys1: int | None = None, k1_token: int = 0, fresh_d0: int = 0, want_stats: bool = False,
                    leave_parts: bool = False, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                   keep_first: int | None = None, chunk: int | None = None, softcap: float | None = None):
+                   keep_first: int | None = None, chunk: int | None = None, softcap: float | None = None, gate_per_head: bool = False,
+                   differential: "DifferentialMaps | None" = None, turn: torch.Tensor | None = None, turn_neighbours: bool = False,
+                   out: torch.Tensor | None = None):
     """Attention in its general form: queries ``q0 [N, H, d0]`` and optionally ``q1 [N, H, d1]`` (lanes behind q0's),
     keys and values addressed by ``(page, head, token)`` strides in elements, an optional bias ``-slopes[h] * distance``.
     Returns ``[N, H, value_dim]``.
@@ -1080,14 +1119,27 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
     no value.  ``gate`` (float32 ``[N, >= H * value_dim]``, rows may have a pitch): the output is multiplied by its sigmoid.
     ``keep_first``: with a window, the keys at positions below it stay visible to every later query.  ``chunk``: a query sees
     only the keys of its own block of so many positions, counted from 0.  ``softcap``: a scaled score s becomes
-    ``softcap * tanh(s / softcap)`` before the distance bias is taken off."""
-    n, d0 = q0.shape[0], q0.shape[2]
+    ``softcap * tanh(s / softcap)`` before the distance bias is taken off.  ``gate_per_head``: one gate a head, ``gate [N, >= H]``.
+    ``differential`` (a :class:`DifferentialMaps`): ``q0 [N, H, 2 * d]`` holds two queries a head side by side, key rows likewise;
+    each has a softmax over the same values and the head's output is the norm of their difference.  ``turn`` (float32
+    ``[N, value_dim / 2, 2]``, cosines and sines): pair m of a head's output, lanes m and m + value_dim/2 (``turn_neighbours``:
+    2m and 2m + 1), is turned back by the token's angle (the values were cached turned by theirs).  ``out``: where the result
+    goes, ``[N, H, value_dim]`` with any token stride."""
+    maps = 2 if differential is not None else 1
+    n, d0 = q0.shape[0], q0.shape[2] // maps
+    _need(q0.shape[2] == maps * d0, "attention_rows: two maps a head have queries of an even number of lanes")
+    _need(maps == 1 or (q1 is None and sinks is None and not key_part and not want_stats and not leave_parts), "two maps a head: plain queries, a whole softmax, no sinks")
+    _need(turn is None or (turn.dtype == torch.float32 and turn.is_contiguous() and value_dim % 2 == 0 and tuple(turn.shape) == (n, value_dim // 2, 2)
+                           and not key_part and not want_stats and not leave_parts), "turn: float32 [N, value_dim / 2, 2], for a whole softmax")
+    diff = (differential.weight, differential.eps, differential.scale) if differential is not None else (0.0, 0.0, 0.0)
+    more = (int(gate_per_head), maps, d0, d0, *(float(v) for v in diff), _ptr(turn), int(turn_neighbours))
     keep_first, chunk, softcap = int(keep_first or 0) if window else 0, int(chunk or 0), float(softcap or 0.0)
     _need(keep_first >= 0 and chunk >= 0 and softcap >= 0.0, "attention_rows: keep_first, chunk and softcap are not negative")
     if sinks is not None:
         _need(sinks.dtype == torch.float32 and sinks.numel() == num_heads and sinks.is_contiguous(), "sinks must be float32 [heads]")
     if gate is not None:
-        _need(gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape[0] == n and gate.shape[1] >= num_heads * value_dim, "the gate must be float32 [N, heads * value_dim]")
+        _need(gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape[0] == n
+              and gate.shape[1] >= num_heads * (1 if gate_per_head else value_dim), "the gate must be float32 [N, heads * value_dim] (or [N, heads])")
         _need(not leave_parts, "a gate is applied where the output is written, not to partial results")
     gate_token = 0 if gate is None else gate.stride(0)
     d1 = 0 if q1 is None else q1.shape[2]
@@ -1095,7 +1147,9 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
     _i32(page_table, "page_table")
     if slopes is not None:
         _need(slopes.dtype == torch.float32 and slopes.numel() == num_heads and slopes.is_contiguous(), "slopes must be float32 [heads]")
-    out = torch.empty((n, num_heads, value_dim), dtype=q0.dtype, device=q0.device)
+    if out is None:
+        out = torch.empty((n, num_heads, value_dim), dtype=q0.dtype, device=q0.device)
+    _need(tuple(out.shape) == (n, num_heads, value_dim) and out.dtype == q0.dtype and out.stride(2) == 1, "attention_rows: out [N, H, value_dim]")
     if q0.dtype == torch.bfloat16 and not _FORCE_GENERIC_ATTENTION and d0 % 16 == 0 and d1 % 16 == 0 and value_dim % 16 == 0 and value_dim <= 256:
         # the tensor cores: 64 rows of (token, group member) a CTA; few CTAs and long contexts: the keys cut over several
         group = num_heads // num_kv_heads
@@ -1104,15 +1158,15 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
             longest = min(longest, window + keep_first + ctx.max_query_len)
         if chunk:
             longest = min(longest, chunk + ctx.max_query_len)
-        ctas = -(-ctx.max_query_len * group // 64) * num_kv_heads * ctx.num_requests
-        splits = max(1, min(-(-longest // 256), _sm_count() // ctas, 16, _SPLIT_SCRATCH_BYTES // (n * num_heads * value_dim * 4)))
+        ctas = -(-ctx.max_query_len * group * maps // 64) * num_kv_heads * ctx.num_requests
+        splits = max(1, min(-(-longest // 256), _sm_count() // ctas, 16, _SPLIT_SCRATCH_BYTES // (n * num_heads * maps * value_dim * 4)))
         if key_part or want_stats:
             splits = 1
         stats = torch.empty((n, num_heads, 2), dtype=torch.float32, device=q0.device) if want_stats else None
         part_o = part_ml = None
         if splits > 1:
-            part_o = torch.empty((n * num_heads * splits * value_dim,), dtype=torch.float32, device=q0.device)
-            part_ml = torch.empty((n * num_heads * splits * 2,), dtype=torch.float32, device=q0.device)
+            part_o = torch.empty((n * num_heads * maps * splits * value_dim,), dtype=torch.float32, device=q0.device)
+            part_ml = torch.empty((n * num_heads * maps * splits * 2,), dtype=torch.float32, device=q0.device)
         code = _launch(
             "llm_attention_rows_mma", _ptr(q0), q0.stride(0), q0.stride(1), d0, _ptr(q1), 0 if q1 is None else q1.stride(0),
             0 if q1 is None else q1.stride(1), d1, None if (leave_parts and splits > 1) else _ptr(out), out.stride(0), out.stride(1),
@@ -1120,7 +1174,7 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
             value_dim, _ptr(page_table), page_table.shape[1], _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.context_lens),
             _ptr(slopes), n, ctx.num_requests, ctx.max_query_len, num_heads, num_kv_heads, page_size, int(window or 0), float(scale),
             splits, _ptr(part_o), _ptr(part_ml), int(key_part), keys1, int(k1_token), int(fresh_d0), _ptr(stats), _ptr(sinks), _ptr(gate),
-            gate_token, keep_first, chunk, softcap, _stream(),
+            gate_token, keep_first, chunk, softcap, *more, _stream(),
         )
         if code != 10002:
             _check(code, "attention_rows (tensor cores)")
@@ -1135,10 +1189,18 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
         0 if q1 is None else q1.stride(1), d1, _ptr(out), out.stride(0), out.stride(1), keys, *k_strides, values, *v_strides,
         value_dim, _code(q0.dtype), _ptr(page_table), page_table.shape[1], _ptr(ctx.token_request), _ptr(ctx.cu_tokens),
         _ptr(ctx.context_lens), _ptr(slopes), n, num_heads, num_kv_heads, page_size, int(window or 0), float(scale), _ptr(sinks),
-        _ptr(gate), gate_token, keep_first, chunk, softcap, _stream(),
+        _ptr(gate), gate_token, keep_first, chunk, softcap, *more, _stream(),
     )
     _check(code, "attention_rows")
     return out
+
+
+class DifferentialMaps:
+    """How the outputs a1 and a2 of a head's two score maps become one: ``u = a1 - weight * a2``, then
+    ``u / sqrt(mean(u^2) + eps) * scale`` over the head's lanes."""
+
+    def __init__(self, weight: float, eps: float, scale: float):
+        self.weight, self.eps, self.scale = float(weight), float(eps), float(scale)
 
 
 class AttentionParts:
@@ -1240,22 +1302,32 @@ def biased_paged_attention(qkv: torch.Tensor, pool: torch.Tensor, page_table: to
 def paged_softmax_attention(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor, ctx, *, num_heads: int, num_kv_heads: int,
                             key_dim: int, value_dim: int, scale: float, window: int | None = None, sinks: torch.Tensor | None = None,
                             gate: torch.Tensor | None = None, keep_first: int | None = None, chunk: int | None = None,
-                            softcap: float | None = None, slopes: torch.Tensor | None = None) -> torch.Tensor:
+                            softcap: float | None = None, slopes: torch.Tensor | None = None, gate_per_head: bool = False,
+                            differential: DifferentialMaps | None = None, turn: torch.Tensor | None = None, turn_neighbours: bool = False,
+                            out: torch.Tensor | None = None) -> torch.Tensor:
     """Grouped-query softmax attention of prepared queries ``q [N, num_heads * key_dim]`` over keys and values in
     ``pool [pages, 2, kv_heads, page_size, D]`` (``D >= key_dim, value_dim``), with an optional sink per head and an
     optional sigmoid gate on the output, a window that may keep the first keys, blocks of positions, a cap on the scores and a
-    distance bias per head (see :func:`attention_rows`).  Returns ``[N, num_heads * value_dim]``."""
-    _need(q.dim() == 2 and q.stride(1) == 1 and q.shape[1] == num_heads * key_dim, "paged_softmax_attention: q [N, heads * key_dim]")
+    distance bias per head, one gate a head, two score maps a head (``key_dim`` lanes each, queries and key rows side by side)
+    and values that turn back (see :func:`attention_rows`).  ``out``: where the result goes, ``[N, num_heads * value_dim]`` whose
+    rows may have a pitch.  Returns ``[N, num_heads * value_dim]``."""
+    key_dim = key_dim * (2 if differential is not None else 1)
+    _need(q.dim() == 2 and q.stride(1) == 1 and q.shape[1] == num_heads * key_dim, "paged_softmax_attention: q [N, heads * key_dim (times two for two maps)]")
     _need(pool.dtype == q.dtype and pool.is_contiguous() and pool.dim() == 5 and tuple(pool.shape[1:3]) == (2, num_kv_heads), "the pool plane does not match the heads")
     page_size, row = pool.shape[3], pool.shape[4]
     _need(row >= max(key_dim, value_dim), "the pool's rows are shorter than a key or a value")
     q3 = q.as_strided((q.shape[0], num_heads, key_dim), (q.stride(0), key_dim, 1), q.storage_offset())
     head, page = page_size * row, 2 * num_kv_heads * page_size * row
     values = pool.data_ptr() + num_kv_heads * head * pool.element_size()
-    out = attention_rows(q3, None, _ptr(pool), (page, head, row), values, (page, head, row), value_dim, page_table, page_size, ctx,
-                         num_heads=num_heads, num_kv_heads=num_kv_heads, scale=scale, window=window, sinks=sinks, gate=gate,
-                         keep_first=keep_first, chunk=chunk, softcap=softcap, slopes=slopes)
-    return out.view(q.shape[0], num_heads * value_dim)
+    if out is not None:
+        _need(out.dim() == 2 and tuple(out.shape) == (q.shape[0], num_heads * value_dim) and out.stride(1) == 1 and out.dtype == q.dtype,
+              "paged_softmax_attention: out [N, heads * value_dim] of the queries' type")
+    o3 = None if out is None else out.as_strided((q.shape[0], num_heads, value_dim), (out.stride(0), value_dim, 1), out.storage_offset())
+    done = attention_rows(q3, None, _ptr(pool), (page, head, row), values, (page, head, row), value_dim, page_table, page_size, ctx,
+                          num_heads=num_heads, num_kv_heads=num_kv_heads, scale=scale, window=window, sinks=sinks, gate=gate,
+                          keep_first=keep_first, chunk=chunk, softcap=softcap, slopes=slopes, gate_per_head=gate_per_head,
+                          differential=differential, turn=turn, turn_neighbours=turn_neighbours, out=o3)
+    return done.view(q.shape[0], num_heads * value_dim) if out is None else out
 
 
 def head_prepare(proj: torch.Tensor, positions: torch.Tensor | None, *, heads: int, kv_heads: int, dim: int, value_dim: int = 0,
@@ -1263,7 +1335,8 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor | None, *, heads: i
                  eps: float = 0.0, freq: torch.Tensor | None = None, warm: tuple[float, int] | None = None,
                  values_are_keys: bool = False, pool: torch.Tensor | None = None, slot_map: torch.Tensor | None = None,
                  out_dtype: torch.dtype | None = None, interleaved: bool = False, values_out: torch.Tensor | None = None,
-                 values_first: torch.Tensor | None = None, values_lambda: float = 0.0) -> torch.Tensor:
+                 values_first: torch.Tensor | None = None, values_lambda: float = 0.0, norm_whole: bool = False, maps: int = 1,
+                 value_freq: torch.Tensor | None = None, turn_out: torch.Tensor | None = None) -> torch.Tensor:
     """From a token's stacked projections ``proj`` rows ``[heads x dim | kv_heads x dim | kv_heads x value_dim]`` to
     queries, keys and values, in this order: ``bias`` (float32, laid out like the row) is added; with ``q_weight`` /
     ``k_weight`` (float32 ``[dim]``) every head is RMS-normed over its lanes (``eps`` inside the root) and weighted; with
@@ -1274,38 +1347,48 @@ def head_prepare(proj: torch.Tensor, positions: torch.Tensor | None, *, heads: i
     ``interleaved``: the rotated lanes pair as ``(2i, 2i + 1)``.  ``values_out`` (float32 ``[N, kv_heads * value_dim]``)
     takes the values as projected, bias included; with ``values_first`` (the same shape: what an earlier layer kept for
     these tokens) the values become ``(1 - values_lambda) v + values_lambda values_first`` on their way to the pool.
+    ``norm_whole``: all query heads are normed together as one vector, all key heads as another (``q_weight [heads * dim]``,
+    ``k_weight [kv_heads * dim]``).  ``maps = 2``: every two key heads in a row share a value head and a row of the pool, side by
+    side (``kv_heads`` counts the keys; the values, and the pool's heads, are half as many).  ``value_freq`` (float32
+    ``[value_dim / 2]``): every value head's pairs ``(m, m + value_dim/2)`` (``interleaved``: ``(2m, 2m + 1)``) turn by
+    ``position * value_freq[m]`` on their way to the pool; ``turn_out`` (float32 ``[N, value_dim / 2, 2]``) takes the cosines and sines.
     Returns the queries ``[N, heads * dim]`` in ``out_dtype`` (default: the pool's type)."""
-    cols = (heads + kv_heads) * dim + (0 if values_are_keys else kv_heads * value_dim)
+    _need(maps in (1, 2) and kv_heads % maps == 0, "head_prepare: one or two keys a value head")
+    value_heads = kv_heads // maps
+    cols = (heads + kv_heads) * dim + (0 if values_are_keys else value_heads * value_dim)
     _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] >= cols, "head_prepare: proj rows are too short")
     n = proj.shape[0]
     rot = 0
     if freq is not None:
         _need(freq.dtype == torch.float32 and freq.is_contiguous(), "head_prepare: freq is float32")
         rot = 2 * freq.numel()
-    if rot or warm:
+    if rot or warm or value_freq is not None:
         _i32(positions, "positions")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == cols, "head_prepare: the bias is float32, laid out like the row")
-    normed = q_weight is not None
-    for w in (q_weight, k_weight):
-        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == dim), "head_prepare: norm weights are float32 [dim]")
+    normed = 0 if q_weight is None else 2 if norm_whole else 1
+    for w, count in ((q_weight, heads), (k_weight, kv_heads)):
+        _need(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == dim * (count if norm_whole else 1)), "head_prepare: norm weights are float32 [dim] (or of the whole projection)")
+    if value_freq is not None:
+        _need(value_freq.dtype == torch.float32 and value_freq.is_contiguous() and 2 * value_freq.numel() == value_dim, "head_prepare: value_freq is float32 [value_dim / 2]")
+        _need(turn_out is None or (turn_out.dtype == torch.float32 and turn_out.is_contiguous() and tuple(turn_out.shape) == (n, value_dim // 2, 2)), "head_prepare: turn_out is float32 [N, value_dim / 2, 2]")
     if kv_heads:
-        _need(pool is not None and pool.is_contiguous() and pool.dim() == 5 and tuple(pool.shape[1:3]) == (2, kv_heads), "the pool plane does not match the heads")
+        _need(pool is not None and pool.is_contiguous() and pool.dim() == 5 and tuple(pool.shape[1:3]) == (2, value_heads), "the pool plane does not match the heads")
         _need(not normed or k_weight is not None, "head_prepare: normed keys need a weight")
         _i32(slot_map, "slot_map")
         out_dtype = pool.dtype
     out_dtype = out_dtype or proj.dtype
     for t in (values_out, values_first):
-        _need(t is None or (kv_heads and not values_are_keys and t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == (n, kv_heads * value_dim)),
+        _need(t is None or (kv_heads and not values_are_keys and t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == (n, value_heads * value_dim)),
               "head_prepare: the values kept for, or taken from, another layer are float32 [N, kv_heads * value_dim]")
     q = torch.empty((n, heads * dim), dtype=out_dtype, device=proj.device)
     coef, every = (float(warm[0]), int(warm[1])) if warm else (0.0, 0)
     code = _launch(
         "llm_head_prepare", _ptr(proj), _code(proj.dtype), proj.stride(0), _ptr(bias), _ptr(q), q.stride(0), _ptr(pool) if kv_heads else None,
         _code(out_dtype), _ptr(slot_map) if kv_heads else None, pool.shape[3] if kv_heads else 1, pool.shape[4] if kv_heads else dim,
-        _ptr(q_weight), _ptr(k_weight), float(eps), int(normed), _ptr(freq), rot, _ptr(positions) if (rot or warm) else None, coef, every,
+        _ptr(q_weight), _ptr(k_weight), float(eps), int(normed), _ptr(freq), rot, _ptr(positions) if (rot or warm or value_freq is not None) else None, coef, every,
         n, heads, kv_heads, dim, value_dim, int(values_are_keys), int(interleaved), _ptr(values_out), _ptr(values_first), float(values_lambda),
-        _stream(),
+        maps, _ptr(value_freq), _ptr(turn_out), _stream(),
     )
     _check(code, "head_prepare")
     return q

@@ -105,6 +105,10 @@ class Part:
     # step through this part can be captured in a CUDA graph.  A captured step's first run is an
     # ordinary pass and every later one a replay, so each step runs exactly once.
     graph_safe = False
+    # True if the part ends in a plain product of a matrix that a block may run itself, together with another part's: then
+    # ``output_width`` is the inner size of that product, ``release_output_matrix()`` hands the matrix ``[hidden, output_width]``
+    # over (once, after ``bind``), and ``forward(..., into=view)`` leaves the product's input rows in ``view [N, output_width]``.
+    joins_output = False
 
     def tensors(self) -> dict[str, TensorSpec]:
         return {}

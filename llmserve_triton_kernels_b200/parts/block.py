@@ -13,7 +13,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import Block, FeedForward, Mixer, Norm, register_part
+from .base import Block, CompositeSpec, FeedForward, Mixer, Norm, StateSpec, TensorSpec, register_part
 
 
 def _takes_factored(part) -> bool:
@@ -111,6 +111,99 @@ class MixerOnlyBlock(PreNormBlock):
         return self._scaled(self.mixer.forward(x, ctx, cache, sink=sink) if sink else self.mixer.forward(x, ctx, cache))
 
 
+class ParallelBlock(PreNormBlock):
+    """Mixer and feed-forward side by side, each behind a norm of its own of the same rows, with an optional token shift on what
+    the mixer reads:
+
+        h = norm1(x),  h_t <- h_t + shift * (h_(t-1) - h_t)          (``token_shift``: a tensor ``shift [hidden]`` of this block)
+        x <- x + mixer(h) + feed_forward(norm2(x))
+
+    ``h_(t-1)`` is the unshifted h of the token in front in the same request (zeros in front of the first); the last one of every
+    step is kept in a 32-bit state slot beside what the mixer keeps.  Both norms, the shift and the slot are one kernel.  Where
+    both parts end in a plain product (``joins_output``) the block stacks the two matrices side by side and runs one product
+    that adds both contributions into the stream."""
+
+    accepts_sink = True  # the joined product's end may add into the stream
+
+    def __init__(self, mixer_norm: Norm, mixer: Mixer, ff_norm: Norm | None, feed_forward: FeedForward | None, hidden_size: int,
+                 token_shift: bool = False, shift_name: str = "shift"):
+        self.mixer_norm, self.mixer, self.ff_norm, self.feed_forward = mixer_norm, mixer, ff_norm, feed_forward
+        self.hidden_size, self.token_shift, self.shift_name = int(hidden_size), bool(token_shift), shift_name
+        self.residual_scale = 1.0
+        # two norms read the rows, and a shifted row is no multiple of one row: nobody in front can hand the stream on normalised
+        mixer_norm.feeds_factored = False
+        self.shift: torch.Tensor | None = None
+        self.w_join: torch.Tensor | None = None  # [hidden, mixer's inner size + feed-forward's]
+
+    def owned_parts(self):
+        return [p for p in (self.mixer_norm, self.mixer, self.ff_norm, self.feed_forward) if p is not None]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for p in self.owned_parts())
+
+    def tensors(self):
+        return {self.shift_name: TensorSpec((self.hidden_size,), init="half_plus_normal")} if self.token_shift else {}
+
+    def bind(self, tensors, dtype, device) -> None:
+        """Called after the parts' own ``bind``."""
+        if self.token_shift:
+            self.shift = tensors[self.shift_name].to(device=device, dtype=torch.float32).contiguous()
+        ends = [p for p in (self.mixer, self.feed_forward) if p is not None]
+        if all(p.joins_output for p in ends):
+            self.w_join = torch.cat([p.release_output_matrix() for p in ends], dim=1).contiguous()
+
+    def cache_spec(self):
+        spec = self.mixer.cache_spec()
+        if not self.token_shift:
+            return spec
+        parts = spec.parts if isinstance(spec, CompositeSpec) else (spec,)
+        return CompositeSpec((*parts, StateSpec((self.hidden_size,), torch.float32)))
+
+    def _views(self, cache):
+        """``(the mixer's view, the state slots of the shift or None)``."""
+        if not self.token_shift:
+            return cache, None
+        *mine, state = cache.parts
+        return (type(cache)(mine) if isinstance(self.mixer.cache_spec(), CompositeSpec) else mine[0]), state
+
+    def forward(self, resid, pending, ctx, cache, next_norm=None):
+        delta, alpha = ops.split_pending(pending)
+        if delta is not None:
+            ops.stream_inject(resid, delta, alpha)
+        view, state = self._views(cache)
+        h, g = self.mixer_norm.pair_forward(resid, self.ff_norm, ctx, self.shift, None if state is None else state.states,
+                                            None if state is None else state.slots)
+        if self.w_join is None:
+            y = self.mixer.forward(h, ctx, view)
+            if self.feed_forward is None:
+                return y
+            delta, alpha = ops.split_pending(y)
+            z = self.feed_forward.forward(g, ctx)
+            ops.stream_inject(resid, delta, alpha)
+            return z
+        width = self.mixer.output_width
+        rows = torch.empty((h.shape[0], self.w_join.shape[1]), dtype=h.dtype, device=h.device)
+        self.mixer.forward(h, ctx, view, into=rows[:, :width])
+        if self.feed_forward is not None:
+            self.feed_forward.forward(g, ctx, into=rows[:, width:])
+        sink = self._sink(self, next_norm, resid, ctx)
+        if sink is not None:
+            handed_on = sink.linear(rows, self.w_join)
+            if handed_on is not None:
+                return handed_on
+        return ops.linear(rows, self.w_join, out_dtype=torch.float32)
+
+
+class ParallelMixerOnlyBlock(ParallelBlock):
+    """The same without a feed-forward: ``x <- x + mixer(h)``."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer"}
+
+    def __init__(self, mixer_norm: Norm, mixer: Mixer, hidden_size: int, token_shift: bool = False, shift_name: str = "shift"):
+        super().__init__(mixer_norm, mixer, None, None, hidden_size, token_shift, shift_name)
+
+
 class HyperConnectionBlock(Block):
     """A pre-norm layer over a residual stream kept in S copies ``x_1 .. x_S`` (hyper-connections).  For each of its parts
     q (1: the mixer, 2: the feed-forward) it owns ``hc<q>.in [S]``, ``hc<q>.out [S]`` and ``hc<q>.mix [S, S]``:
@@ -142,8 +235,6 @@ class HyperConnectionBlock(Block):
         return 1 if self.feed_forward is None else 2
 
     def tensors(self):
-        from .base import TensorSpec
-
         S, specs = self.streams, {}
         for name in self.names[: self._parts()]:
             specs[f"{name}.in"] = TensorSpec((S,), init="ones_plus_normal")
@@ -181,5 +272,7 @@ class HyperConnectionMixerOnlyBlock(HyperConnectionBlock):
 
 register_part("block", "hyper_connection", HyperConnectionBlock)
 register_part("block", "hyper_connection_mixer_only", HyperConnectionMixerOnlyBlock)
+register_part("block", "parallel", ParallelBlock)
+register_part("block", "parallel_mixer_only", ParallelMixerOnlyBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "pre_norm_mixer_only", MixerOnlyBlock)

@@ -73,12 +73,13 @@ register_part("feed_forward", "gated_mlp", GatedMLP)
 
 
 class DenseMLP(FeedForward):
-    """``down(act(up(x)))`` without biases; ``act`` one of ``relu2`` (the square of relu), ``gelu_tanh``, ``silu``.
-    ``tensor_names``: local names of the two matrices (default ``up`` and ``down``)."""
+    """``down(act(up(x)))`` without biases; ``act`` one of ``relu2`` (the square of relu), ``gelu_tanh``, ``gelu`` (the erf
+    form), ``silu``.  ``tensor_names``: local names of the two matrices (default ``up`` and ``down``)."""
 
     graph_safe = True
     accepts_sink = True
-    activations = ("relu2", "gelu_tanh", "silu")
+    joins_output = True
+    activations = ("relu2", "gelu_tanh", "silu", "gelu")
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu2", tensor_names: dict[str, str] | None = None):
         if activation not in self.activations:
@@ -96,8 +97,18 @@ class DenseMLP(FeedForward):
         self.w_up = tensors[self.names["up"]].to(device=device, dtype=dtype).contiguous()
         self.w_down = tensors[self.names["down"]].to(device=device, dtype=dtype).contiguous()
 
-    def forward(self, x, ctx, sink=None):
-        act = ops.linear_act(x, self.w_up, self.activation)
+    @property
+    def output_width(self) -> int:
+        return self.intermediate_size
+
+    def release_output_matrix(self) -> torch.Tensor:
+        w, self.w_down = self.w_down, None
+        return w
+
+    def forward(self, x, ctx, sink=None, into=None):
+        act = ops.linear_act(x, self.w_up, self.activation, out=into)
+        if into is not None:
+            return None
         if sink is not None:
             handed_on = sink.linear(act, self.w_down)
             if handed_on is not None:
@@ -130,12 +141,13 @@ class RoutedMLP(FeedForward):
 
     graph_safe = True
     accepts_sink = True
+    activations = ("relu2", "gelu_tanh", "silu")
 
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, activation: str = "relu2",
                  router_scale: float = 1.0, correction: bool = True, renormalize: bool = False, shared_size: int | None = None,
                  shared_gate: bool = True):
-        if activation not in DenseMLP.activations:
-            raise ValueError(f"activation {activation!r} is not built; known: {DenseMLP.activations}")
+        if activation not in self.activations:
+            raise ValueError(f"activation {activation!r} is not built; known: {self.activations}")
         if not 1 <= int(top) <= int(experts):
             raise ValueError(f"a token uses {top} of {experts} experts")
         self.hidden_size, self.experts, self.top, self.expert_size = int(hidden_size), int(experts), int(top), int(expert_size)

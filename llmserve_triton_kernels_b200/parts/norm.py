@@ -53,6 +53,14 @@ class RMSNorm(Norm):
             return None
         return ops.branch_sum_rmsnorm(pending, resid, self.weight, self.eps, self.out_dtype)
 
+    def pair_forward(self, resid, other: "RMSNorm | None", ctx, shift=None, states=None, state_slots=None):
+        """This norm and ``other`` (None: this one alone) of the same rows in one kernel, this one's result passed through a token
+        shift where there is one (see ``ops.shift_norm``): ``(shifted, other's or None)``."""
+        if self.groups != 1 or (other is not None and (other.groups != 1 or other.eps != self.eps)):
+            raise NotImplementedError("two norms of the same rows are built for plain RMS norms of one eps")
+        return ops.shift_norm(resid, self.weight, self.eps, w2=None if other is None else other.weight, shift=shift, states=states,
+                              ctx=ctx, state_slots=state_slots, out_dtype=self.out_dtype)
+
     def add_streams(self, streams, update, read_in, rows=None):
         """For a residual stream kept in several copies (``streams [S, N, size]``): the copies take up ``update`` (an
         ``ops.StreamUpdate`` or None) in place, are read in with the weights ``read_in [S]`` (None: summed) and the result

@@ -29,12 +29,14 @@ _NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": 
 
 def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> torch.Tensor:
     """``f_i = base^(-2i / dims)`` for ``i < dims / 2`` (float64 on the host, rounded to float32 once), with long
-    wavelengths stretched as ``scaling`` says."""
+    wavelengths stretched as ``scaling`` says; a ``scaling`` of a ``factor`` alone divides every frequency by it."""
     if dims % 2:
         raise ValueError(f"rotated lanes come in pairs, got {dims}")
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = float(base) ** (-2.0 * i / max(dims, 1))
-    if scaling:
+    if scaling and set(scaling) == {"factor"}:
+        f = f / float(scaling["factor"])
+    elif scaling:
         factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         wavelength = 2.0 * math.pi / f
         t = (original / wavelength - low) / (high - low) if high != low else torch.ones_like(f)

@@ -6,9 +6,12 @@
                      y_t = sum_j w[:, j] u_(t - taps + 1 + j) with weights ``<name>.conv`` [channels, taps]; a request's last
                      taps - 1 projected rows are kept in a state slot beside its pages
     qk_norm_eps:     every query head and every key head RMS-normed over its lanes, weights ``q.norm`` / ``k.norm`` [dim]
-                     shared by the heads, before rotation
+                     shared by the heads, before rotation (``norm_over = "projection"``: all query heads together as one vector,
+                     all key heads likewise, weights of the projections' sizes)
     rotary:          lanes i and i + dims/2 of the first ``dims`` lanes of every head turn by position * base^(-2i/dims)
-                     (``rotary_layout = "interleaved"``: lanes 2i and 2i + 1)
+                     (``rotary_layout = "interleaved"``: lanes 2i and 2i + 1), divided by ``scaling.factor`` if there is one
+    rotate_values:   the value of position j turns by j, lanes m and m + value_dim/2 (interleaved: 2m and 2m + 1) by
+                     j * base^(-2m/value_dim), and is cached so; a head's output at position i is turned back by i
     value_mix:       "source": the values as projected (bias included, behind the convolution) are handed to later layers of
                      the same pass; "mixed": v <- (1 - vmix) v + vmix v_source, v_source the source layer's values of the same
                      token and ``vmix`` a number of the checkpoint; what is cached is the mixed value
@@ -18,8 +21,12 @@
     distance_bias b: the score then loses slope_h * (i - j), slope_h = 2^(-b (h + 1) / heads)
     keep_first:      with a window, the keys at positions below it stay visible
     chunk:           only the keys of the query's own block of ``chunk`` positions (counted from 0) are visible
+    differential d:  two queries and two keys of ``head_dim`` lanes a head, [map 1, map 2] side by side, over the same values; with
+                     a1, a2 the maps' softmax outputs and w = exp(lq1 . lk1) - exp(lq2 . lk2) + d (``lq1`` ... ``lk2`` [dim], one
+                     number a layer) a head's output is u / sqrt(mean(u^2) + eps) * (1 - d), u = a1 - w a2
     sink:            the softmax's denominator also holds exp(sink_h), a number per head with no key and no value
-    gate:            the heads side by side times sigmoid(W_g x), before the output projection
+    gate:            the heads side by side times sigmoid(W_g x), before the output projection (``gate_per_head``: W_g [heads],
+                     one number a head)
     out = W_o [heads side by side] (+ b_o)
 
 With ``own_kv=False`` the layer has no key and value projections and reads the pages that an earlier entry of the order
@@ -30,6 +37,8 @@ both compute types.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .. import ops
@@ -37,7 +46,7 @@ from .base import CompositeSpec, Mixer, PagedKVSpec, StateSpec, TensorSpec, regi
 from .sigmoid_attention import rotary_frequencies
 
 _NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "g": "g", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "q_norm": "q.norm",
-          "k_norm": "k.norm", "sink": "sink", "o_bias": "o.b", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "value_mix": "vmix"}
+          "k_norm": "k.norm", "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2", "sink": "sink", "o_bias": "o.b", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "value_mix": "vmix"}
 
 
 class SoftmaxAttention(Mixer):
@@ -51,10 +60,11 @@ class SoftmaxAttention(Mixer):
                  window: int | None = None, tensor_names: dict[str, str] | None = None, out_bias: bool = False,
                  rotary_layout: str = "half", keep_first: int | None = None, chunk: int | None = None, softcap: float | None = None,
                  distance_bias: float | None = None, conv: int | None = None, value_mix: str | None = None,
-                 value_mix_key: str = "first_values"):
+                 value_mix_key: str = "first_values", norm_over: str = "head", rotate_values: bool = False,
+                 differential: float | None = None, differential_eps: float = 0.0, gate_per_head: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
-        if not (1 <= int(head_dim) <= 640 and 1 <= int(value_dim) <= 512):
+        if not (1 <= int(head_dim) * (1 if differential is None else 2) <= 640 and 1 <= int(value_dim) <= 512):
             raise ValueError(f"head_dim {head_dim} / value_dim {value_dim}: the kernels take keys of up to 640 and values of up to 512 lanes")
         if values_are_keys and int(value_dim) != int(head_dim):
             raise ValueError(f"values that are the keys have the keys' size {head_dim}, not {value_dim}")
@@ -89,7 +99,22 @@ class SoftmaxAttention(Mixer):
         if value_mix not in (None, "source", "mixed") or (value_mix and (not self.own_kv or self.values_are_keys)):
             raise ValueError(f"value_mix is None, 'source' or 'mixed' for a layer with values of its own, got {value_mix!r}")
         self.value_mix, self.value_mix_key = value_mix, value_mix_key
+        if norm_over not in ("head", "projection"):
+            raise ValueError(f"q and k are normed over each 'head' or over the whole 'projection', not {norm_over!r}")
+        self.norm_whole = norm_over == "projection"
+        self.rotate_values = bool(rotate_values)
+        if self.rotate_values and (not rotary or self.value_dim % 2 or not self.own_kv or self.values_are_keys or self.value_mix):
+            raise ValueError("rotated values need a rotation's base, an even number of lanes, and projections of their own")
+        self.differential = None if differential is None else float(differential)
+        self.differential_eps = float(differential_eps)
+        if self.differential is not None and (not self.own_kv or self.values_are_keys or self.has_sink or self.qk_norm_eps is not None or self.conv):
+            raise ValueError("two score maps a head are built for projections of their own, without norms of q and k, sinks and convolutions")
+        self.maps = 1 if self.differential is None else 2
+        self.gate_per_head = bool(gate_per_head) and self.has_gate
+        self.value_base = float(rotary["base"]) if self.rotate_values else None
+        self.joins_output = not self.out_bias
         self.names = {**_NAMES, **(tensor_names or {})}
+        self.value_freq = self.maps_meet = None
         self.w_in = self.w_out = self.b_in = self.q_weight = self.k_weight = self.sink = self.freq = None
         self.b_out = self.w_conv = self.slopes = None
         self.mix = 0.0
@@ -104,19 +129,22 @@ class SoftmaxAttention(Mixer):
 
     def tensors(self) -> dict[str, TensorSpec]:
         n, H, KV, D, V, hid = self.names, self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size
-        rows = {"q": H * D, "k": KV * D, "v": KV * V}
+        rows = {"q": H * self.maps * D, "k": KV * self.maps * D, "v": KV * V}
         specs = {}
         for role in self._stacked():
             specs[n[role]] = TensorSpec((rows[role], hid))
             if self.bias:
                 specs[n[role + "_bias"]] = TensorSpec((rows[role],))
         if self.has_gate:
-            specs[n["g"]] = TensorSpec((H * V, hid))
+            specs[n["g"]] = TensorSpec((H if self.gate_per_head else H * V, hid))
         specs[n["o"]] = TensorSpec((hid, H * V))
         if self.qk_norm_eps is not None:
-            specs[n["q_norm"]] = TensorSpec((D,), init="ones_plus_normal")
+            specs[n["q_norm"]] = TensorSpec((H * D if self.norm_whole else D,), init="ones_plus_normal")
             if self.own_kv:
-                specs[n["k_norm"]] = TensorSpec((D,), init="ones_plus_normal")
+                specs[n["k_norm"]] = TensorSpec((KV * D if self.norm_whole else D,), init="ones_plus_normal")
+        if self.differential is not None:
+            for role in ("lq1", "lk1", "lq2", "lk2"):
+                specs[n[role]] = TensorSpec((D,))
         if self.has_sink:
             specs[n["sink"]] = TensorSpec((H,))
         if self.out_bias:
@@ -132,6 +160,9 @@ class SoftmaxAttention(Mixer):
         n = self.names
         roles = self._stacked()
         mats = [tensors[n[r]].to(dtype) for r in roles] + ([tensors[n["g"]].to(dtype)] if self.has_gate else [])
+        rows = sum(m.shape[0] for m in mats)
+        if self.gate_per_head and rows % 16:  # a few rows of zeros, so that the stacked product's rows stay on wide boundaries
+            mats.append(torch.zeros((16 - rows % 16, self.hidden_size), dtype=dtype, device=mats[0].device))
         self.w_in = torch.cat(mats, dim=0).to(device).contiguous()
         self.w_out = tensors[n["o"]].to(device=device, dtype=dtype).contiguous()
         f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()  # noqa: E731
@@ -143,7 +174,13 @@ class SoftmaxAttention(Mixer):
         if self.has_sink:
             self.sink = f32(tensors[n["sink"]])
         if self.rotary:
-            self.freq = rotary_frequencies(self.rotary["dims"], self.rotary["base"]).to(device)
+            self.freq = rotary_frequencies(self.rotary["dims"], self.rotary["base"], self.rotary.get("scaling")).to(device)
+        if self.rotate_values:
+            self.value_freq = rotary_frequencies(self.value_dim, self.value_base).to(device)
+        if self.differential is not None:
+            dot = lambda i: float((tensors[n[f"lq{i}"]].double() * tensors[n[f"lk{i}"]].double()).sum())  # noqa: E731
+            weight = math.exp(dot(1)) - math.exp(dot(2)) + self.differential
+            self.maps_meet = ops.DifferentialMaps(weight, self.differential_eps, 1.0 - self.differential)
         if self.out_bias:
             self.b_out = f32(tensors[n["o_bias"]])
         if self.conv:
@@ -160,13 +197,22 @@ class SoftmaxAttention(Mixer):
         return (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim
 
     def cache_spec(self):
-        pages = PagedKVSpec(self.num_kv_heads, max(self.head_dim, self.value_dim), self.window, self.keep_first, self.chunk)
+        pages = PagedKVSpec(self.num_kv_heads, max(self.maps * self.head_dim, self.value_dim), self.window, self.keep_first, self.chunk)
         if self.conv and self.conv > 1:  # the rows that the convolution still reads when the next step begins
             return CompositeSpec((pages, StateSpec((self.conv - 1, self._channels()), torch.float32)))
         return pages
 
-    def forward(self, x, ctx, cache, sink=None, proj=None):
-        """``proj``: the stacked projections (32-bit, rows may have a pitch) where the caller ran the product."""
+    @property
+    def output_width(self) -> int:
+        return self.num_heads * self.value_dim
+
+    def release_output_matrix(self) -> torch.Tensor:
+        w, self.w_out = self.w_out, None
+        return w
+
+    def forward(self, x, ctx, cache, sink=None, proj=None, into=None):
+        """``proj``: the stacked projections (32-bit, rows may have a pitch) where the caller ran the product.  ``into``: the heads
+        side by side go there, and the caller runs the output product."""
         H, KV, D, V = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim
         if proj is None:
             proj = ops.linear(x, self.w_in, out_dtype=torch.float32)
@@ -182,17 +228,24 @@ class SoftmaxAttention(Mixer):
             keep = ctx.shared[self.value_mix_key] = torch.empty((proj.shape[0], KV * V), dtype=torch.float32, device=proj.device)
         elif self.value_mix == "mixed":
             first = ctx.shared[self.value_mix_key]
-        q = ops.head_prepare(proj, ctx.positions, heads=H, kv_heads=kv, dim=D, value_dim=V, bias=self.b_in, q_weight=self.q_weight,
+        turn = None
+        if self.rotate_values:  # the angles' cosines and sines, from the kernel that turns the values to the one that turns the sums back
+            turn = torch.empty((proj.shape[0], V // 2, 2), dtype=torch.float32, device=proj.device)
+        q = ops.head_prepare(proj, ctx.positions, heads=H * self.maps, kv_heads=kv * self.maps, dim=D, value_dim=V, bias=self.b_in, q_weight=self.q_weight,
                              k_weight=self.k_weight, eps=self.qk_norm_eps or 0.0, freq=self.freq, warm=self.q_temp,
                              values_are_keys=self.values_are_keys, pool=cache.pool, slot_map=cache.slot_map, out_dtype=self.dtype,
-                             interleaved=self.rotary_layout == "interleaved", values_out=keep, values_first=first, values_lambda=self.mix)
+                             interleaved=self.rotary_layout == "interleaved", values_out=keep, values_first=first, values_lambda=self.mix,
+                             norm_whole=self.norm_whole, maps=self.maps, value_freq=self.value_freq, turn_out=turn)
         gate = None
         if self.has_gate:
-            start = (H + kv) * D + (0 if self.values_are_keys else kv * V)
-            gate = proj[:, start : start + H * V]
+            start = (H + kv) * self.maps * D + (0 if self.values_are_keys else kv * V)
+            gate = proj[:, start : start + (H if self.gate_per_head else H * V)]
         out = ops.paged_softmax_attention(q, cache.pool, cache.page_table, ctx, num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=V,
                                           scale=self.scale, window=self.window, sinks=self.sink, gate=gate, keep_first=self.keep_first,
-                                          chunk=self.chunk, softcap=self.softcap, slopes=self.slopes)
+                                          chunk=self.chunk, softcap=self.softcap, slopes=self.slopes, gate_per_head=self.gate_per_head,
+                                          differential=self.maps_meet, turn=turn, turn_neighbours=self.rotary_layout == "interleaved", out=into)
+        if into is not None:
+            return None
         if self.b_out is not None:
             return ops.add_bias(ops.linear(out, self.w_out, out_dtype=torch.float32), self.b_out)
         if sink is not None:

@@ -154,12 +154,14 @@ def stream_inject(resid, delta=None, alpha=1.0, ids=None, table=None, vector=Non
         resid.add_(vector)
 
 
-def unary(x, kind, alpha=1.0, inplace=False):
+def unary(x, kind, alpha=1.0, inplace=False, out=None):
     v = x.float()
     if kind == "relu2":
         y = torch.relu(v).pow(2)
     elif kind == "gelu_tanh":
         y = 0.5 * v * (1 + torch.tanh(0.7978845608028654 * (v + 0.044715 * v.pow(3))))
+    elif kind == "gelu":
+        y = 0.5 * v * (1 + torch.erf(v * 0.5**0.5))
     elif kind == "scale":
         y = alpha * v
     elif kind == "silu":
@@ -167,13 +169,15 @@ def unary(x, kind, alpha=1.0, inplace=False):
     else:
         raise ValueError(kind)
     if inplace:
-        x.copy_(y.to(x.dtype))
-        return x
+        out = x
+    if out is not None:
+        out.copy_(y.to(x.dtype))
+        return out
     return y.to(x.dtype)
 
 
-def linear_act(x, w, activation):
-    return unary(linear(x, w), activation, inplace=True)
+def linear_act(x, w, activation, out=None):
+    return unary(linear(x, w), activation, inplace=out is None, out=out)
 
 
 def gate_mul(a, b, kind="sigmoid", per_head=False):
@@ -337,19 +341,39 @@ def biased_paged_attention(qkv, pool, page_table, ctx, *, num_heads, num_kv_head
 
 
 def paged_softmax_attention(q, pool, page_table, ctx, *, num_heads, num_kv_heads, key_dim, value_dim, scale, window=None, sinks=None, gate=None,
-                            keep_first=None, chunk=None, softcap=None, slopes=None):
+                            keep_first=None, chunk=None, softcap=None, slopes=None, gate_per_head=False, differential=None, turn=None,
+                            turn_neighbours=False, out=None):
     H, KV = num_heads, num_kv_heads
     page_size = pool.shape[3]
-    out = torch.empty((q.shape[0], H * value_dim), dtype=q.dtype, device=q.device)
+    maps = 1 if differential is None else 2
+    if out is None:
+        out = torch.empty((q.shape[0], H * value_dim), dtype=q.dtype, device=q.device)
     cu, lens = ctx.cu_tokens.tolist(), ctx.context_lens.tolist()
     for r in range(len(lens)):
         t0, t1, n = cu[r], cu[r + 1], lens[r]
         pages = page_table[r, : -(-n // page_size)].long()
-        k = pool[pages, 0].float().permute(0, 2, 1, 3).reshape(-1, KV, pool.shape[4])[:n, :, :key_dim]
+        k = pool[pages, 0].float().permute(0, 2, 1, 3).reshape(-1, KV, pool.shape[4])[:n, :, : maps * key_dim]
         v = pool[pages, 1].float().permute(0, 2, 1, 3).reshape(-1, KV, pool.shape[4])[:n, :, :value_dim]
         k, v = k.repeat_interleave(H // KV, dim=1), v.repeat_interleave(H // KV, dim=1)
-        o = _attend(q[t0:t1].float().view(t1 - t0, H, key_dim), k, v, n - (t1 - t0), scale, window, slopes, sinks, keep_first, chunk, softcap).reshape(t1 - t0, -1)
-        if gate is not None:
+        qs, ks = q[t0:t1].float().view(t1 - t0, H, maps, key_dim), k.view(n, H, maps, key_dim)
+        o = [_attend(qs[:, :, i], ks[:, :, i], v, n - (t1 - t0), scale, window, slopes, sinks, keep_first, chunk, softcap) for i in range(maps)]
+        if differential is not None:
+            u = o[0] - differential.weight * o[1]
+            o = u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + differential.eps) * differential.scale
+        else:
+            o = o[0]
+        if turn is not None:
+            c, s_ = turn[t0:t1, None, :, 0], turn[t0:t1, None, :, 1]
+            if turn_neighbours:
+                a, b = o[..., 0::2], o[..., 1::2]
+                o = torch.stack((a * c + b * s_, b * c - a * s_), dim=-1).flatten(-2)
+            else:
+                a, b = o[..., : value_dim // 2], o[..., value_dim // 2 :]
+                o = torch.cat((a * c + b * s_, b * c - a * s_), dim=-1)
+        if gate is not None and gate_per_head:
+            o = o * torch.sigmoid(gate[t0:t1, :H].float())[:, :, None]
+        o = o.reshape(t1 - t0, -1)
+        if gate is not None and not gate_per_head:
             o = o * torch.sigmoid(gate[t0:t1, : H * value_dim].float())
         out[t0:t1] = o.to(out.dtype)
     return out
@@ -357,16 +381,19 @@ def paged_softmax_attention(q, pool, page_table, ctx, *, num_heads, num_kv_heads
 
 def head_prepare(proj, positions, *, heads, kv_heads, dim, value_dim=0, bias=None, q_weight=None, k_weight=None, eps=0.0, freq=None,
                  warm=None, values_are_keys=False, pool=None, slot_map=None, out_dtype=None, interleaved=False, values_out=None,
-                 values_first=None, values_lambda=0.0):
+                 values_first=None, values_lambda=0.0, norm_whole=False, maps=1, value_freq=None, turn_out=None):
     n = proj.shape[0]
-    cols = (heads + kv_heads) * dim + (0 if values_are_keys else kv_heads * value_dim)
+    cols = (heads + kv_heads) * dim + (0 if values_are_keys else kv_heads // maps * value_dim)
     row = proj[:, :cols].float()
     if bias is not None:
         row = row + bias.float()
     q = row[:, : heads * dim].view(n, heads, dim)
     k = row[:, heads * dim : (heads + kv_heads) * dim].view(n, kv_heads, dim)
-    v = k if values_are_keys else row[:, (heads + kv_heads) * dim :].view(n, kv_heads, value_dim)
-    if q_weight is not None:
+    v = k if values_are_keys else row[:, (heads + kv_heads) * dim :].view(n, kv_heads // maps, value_dim)
+    if q_weight is not None and norm_whole:
+        whole = lambda x, w: (x.flatten(1) / torch.sqrt(x.flatten(1).pow(2).mean(-1, keepdim=True) + eps) * w.float()).view_as(x)  # noqa: E731
+        q, k = whole(q, q_weight), (whole(k, k_weight) if kv_heads else k)
+    elif q_weight is not None:
         q = q / torch.sqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_weight.float()
         if kv_heads:
             k = k / torch.sqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_weight.float()
@@ -394,9 +421,36 @@ def head_prepare(proj, positions, *, heads, kv_heads, dim, value_dim=0, bias=Non
         out_dtype = pool.dtype
         page_size = pool.shape[3]
         page, off = (slot_map // page_size).long(), (slot_map % page_size).long()
-        pool[page, 0, :, off, :dim] = k.to(pool.dtype)
+        if value_freq is not None:
+            angle = positions.float()[:, None] * value_freq.float()[None, :]
+            if turn_out is not None:
+                turn_out.copy_(torch.stack((angle.cos(), angle.sin()), dim=-1))
+            c, s_ = angle.cos()[:, None, :], angle.sin()[:, None, :]
+            if interleaved:
+                a, b = v[..., 0::2], v[..., 1::2]
+                v = torch.stack((a * c - b * s_, b * c + a * s_), dim=-1).flatten(-2)
+            else:
+                a, b = v[..., : value_dim // 2], v[..., value_dim // 2 :]
+                v = torch.cat((a * c - b * s_, b * c + a * s_), dim=-1)
+        pool[page, 0, :, off, : maps * dim] = k.reshape(n, kv_heads // maps, maps * dim).to(pool.dtype)
         pool[page, 1, :, off, : v.shape[-1]] = v.to(pool.dtype)
     return q.reshape(n, heads * dim).to(out_dtype or proj.dtype)
+
+
+def shift_norm(x, w1, eps, w2=None, shift=None, states=None, ctx=None, state_slots=None, out_dtype=torch.float32):
+    n = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+    h = n * w1
+    first = h
+    if shift is not None:
+        cu, slots = ctx.cu_tokens.tolist(), state_slots.tolist()
+        before = torch.empty_like(h)
+        for r, slot in enumerate(slots):
+            a, b = cu[r], cu[r + 1]
+            before[a] = states[slot]
+            before[a + 1 : b] = h[a : b - 1]
+            states[slot] = h[b - 1]
+        first = h + shift * (before - h)
+    return first.to(out_dtype), None if w2 is None else (n * w2).to(out_dtype)
 
 
 def hyper_mix_norm(streams, update, read_in, weight, eps, rows=None, out_dtype=torch.float32):
@@ -602,6 +656,7 @@ def branch_sum_rmsnorm(pending, resid, weight, eps, out_dtype):
 
 
 ALL = (
+    "shift_norm",
     "short_conv",
     "row_rmsnorm",
     "paged_softmax_attention",
