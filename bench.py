@@ -14,7 +14,7 @@ cache of the live requests) to its time; ``points`` holds decode at batch 1 and 
 Peaks come from MEASURED_PEAKS.json beside this file when present, else from an earlier
 measurement on the same pool (and the line says which).
 
-``python bench.py --design nurolorn-small|nurolorn-1b|kafepel-small|kafepel-1b|nudodra-small|nudodra-1b|tenotar-small|tenotar-1b`` prints, instead of the line, prefill and decode
+``python bench.py --design nurolorn-small|nurolorn-1b|kafepel-small|kafepel-1b|nudodra-small|nudodra-1b|tenotar-small|tenotar-1b|pefedra-small|pefedra-1b`` prints, instead of the line, prefill and decode
 throughput of that configuration beside a Llama of equal width, depth and feed-forward size, and the design's kernels against
 their rooflines.
 
@@ -220,6 +220,7 @@ def design_comparison(args) -> int:
     width, vocab = design["width"], design["vocab"]
     nudodra = design["architecture"] == "Nudodra"
     tenotar = design["architecture"] == "Tenotar"
+    pefedra = design["architecture"] == "Pefedra"
     if nudodra or tenotar:  # no dense feed-forward (or one layer's only): the twin's has the size of what a token uses (its chosen experts and the shared one)
         moe = next(x["mlp"] for x in design["layers"] if x.get("mlp") and x["mlp"].get("kind", "moe") == "moe")
         ff = moe["router"]["top"] * moe["expert"]["ff"] + (moe["shared"]["ff"] if moe.get("shared") else 0)
@@ -260,6 +261,14 @@ def design_comparison(args) -> int:
         compared.insert(1, (args.design.replace("nudodra", "kafepel"), dict(PRESETS[args.design.replace("nudodra", "kafepel")])))
     if tenotar:  # the closest design the engine has: the same softmax attention part and a mixture of gated experts at the same sizes
         compared.insert(1, (args.design.replace("tenotar", "nudodra"), dict(PRESETS[args.design.replace("tenotar", "nudodra")])))
+    if pefedra:  # the closest design the engine has, the same softmax attention part over a window, with a dense feed-forward of as many weights
+        span = design["layers"][0]["mixer"]["mask"]["size"]
+        m = next(x["mixer"] for x in design["layers"] if x["type"] == "attention_2")
+        mixer = {"heads": m["heads"], "kv_heads": m["kv_heads"], "dim": m["dim"], "vdim": m["vdim"], "scale": m["scale"],
+                 "mask": {"size": span, "keep_first": 16}, "rot": {"base": 10000.0, "dims": m["dim"]}}
+        compared.insert(1, ("tenotar-twin", {
+            "architecture": "Tenotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": twin["intermediate_size"]}} for _ in design["layers"]]}))
     for name, cfg_dict in compared:
         a = architecture_of(cfg_dict)
         model = random_model(a.config_class.from_dict(cfg_dict), 0, "bfloat16", device)
@@ -332,8 +341,8 @@ def design_comparison(args) -> int:
 
     bf = torch.bfloat16
     kernels = {}
-    if design["architecture"] in ("Kafepel", "Nudodra", "Tenotar"):
-        (_tenotar_kernels if tenotar else _nudodra_kernels if nudodra else _kafepel_kernels)(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device)
+    if design["architecture"] in ("Kafepel", "Nudodra", "Tenotar", "Pefedra"):
+        (_pefedra_kernels if pefedra else _tenotar_kernels if tenotar else _nudodra_kernels if nudodra else _kafepel_kernels)(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device)
         out["kernels"] = kernels
         out["peaks"] = {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"]}
         print(json.dumps(out, indent=1))
@@ -669,6 +678,96 @@ def _tenotar_kernels(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor,
         hbm(f"nudodra_expert_gated_act_{label}", us, n * ((top * eff + sff) * 4 + (E * eff + sff) * 2))
 
 
+def _pefedra_kernels(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device) -> None:
+    """The Pefedra design's own kernels, alone, at the preset's sizes: one request of 2,048 prompt tokens, and 8 decoding requests of
+    2,048 cached tokens; beside each the like kernel of the Tenotar design (the closest one the engine has) at the same sizes.
+    Attention's arithmetic counts the (query, key) pairs that the window leaves, two maps' for the heads that have two; a decode
+    step's bytes are the cached rows that it leaves."""
+    bf = torch.bfloat16
+    A = next(x["mixer"] for x in design["layers"] if x["type"] == "attention")
+    B = next(x["mixer"] for x in design["layers"] if x["type"] == "attention_2")
+    width, ff = design["width"], next(x["mlp"]["ff"] for x in design["layers"] if x.get("mlp"))
+    window = A["mask"]["size"]
+
+    def seen(qs, cs):
+        return sum(min(p + 1, window) for q, c in zip(qs, cs) for p in range(c - q, c))
+
+    for label, qs, cs in (("prefill_2048", [2048], [2048]), ("decode_8x2048", [1] * 8, [2048] * 8)):
+        ctx, table, slots, pages = ctx_for(qs, cs)
+        n, prefill, pairs = ctx.num_tokens, label.startswith("prefill"), seen(qs, cs)
+
+        def attention(name, H, KV, D, V, maps, like=None, **more):
+            pool = torch.randn(pages, 2, KV, 16, max(maps * D, V), device=device).to(bf)
+            q = (torch.randn(n, H * maps * D, device=device) * 0.3).to(bf)
+            us = timed(lambda: ops.paged_softmax_attention(q, pool, table, ctx, num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=V, scale=D ** -0.5,
+                                                           window=window, **more))
+            work = 2.0 * pairs * H * maps * (D + V) if prefill else pairs * KV * (maps * D + V) * 2 + n * H * (maps * D + V) * 2
+            (tensor if prefill else hbm)(f"{name}_{label}", us, work, like=like)
+
+        gate = torch.randn(n, B["heads"], device=device)
+        turn = torch.rand(n, B["vdim"] // 2, 2, device=device)
+        attention("two_map_attention", A["heads"], A["kv_heads"], A["dim"], A["vdim"], 2, like="tenotar_window_attention",
+                  differential=ops.DifferentialMaps(0.5, 1e-6, 0.5))
+        attention("turned_value_attention", B["heads"], B["kv_heads"], B["dim"], B["vdim"], 1, like="tenotar_window_attention", turn=turn, gate=gate,
+                  gate_per_head=True)
+        attention("tenotar_window_attention", B["heads"], B["kv_heads"], B["dim"], B["vdim"], 1, keep_first=16)
+
+        def prepare(name, H, KV, D, V, maps, like=None, **more):
+            cols = (H + KV) * maps * D + KV * V
+            pool = torch.zeros(pages, 2, KV, 16, max(maps * D, V), device=device, dtype=bf)
+            proj, bias = torch.randn(n, cols, device=device), torch.randn(cols, device=device)
+            us = timed(lambda: ops.head_prepare(proj, ctx.positions, heads=H * maps, kv_heads=KV * maps, dim=D, value_dim=V, bias=bias, pool=pool,
+                                                slot_map=slots, maps=maps, **more))
+            hbm(f"{name}_{label}", us, n * cols * 6, like=like)
+
+        qw, kw = torch.ones(B["heads"] * B["dim"], device=device), torch.ones(B["kv_heads"] * B["dim"], device=device)
+        prepare("head_prepare_two_maps", A["heads"], A["kv_heads"], A["dim"], A["vdim"], 2, like="tenotar_head_prepare", freq=torch.rand(A["rot"]["dims"] // 2, device=device))
+        prepare("head_prepare_turned_values", B["heads"], B["kv_heads"], B["dim"], B["vdim"], 1, like="tenotar_head_prepare", q_weight=qw, k_weight=kw, eps=1e-6,
+                norm_whole=True, freq=torch.rand(B["rot"]["dims"] // 2, device=device), value_freq=torch.rand(B["vdim"] // 2, device=device), turn_out=turn)
+        prepare("tenotar_head_prepare", B["heads"], B["kv_heads"], B["dim"], B["vdim"], 1, q_weight=qw[: B["dim"]].contiguous(), k_weight=kw[: B["dim"]].contiguous(),
+                eps=1e-6, freq=torch.rand(B["dim"] // 2, device=device), interleaved=True)
+        # the two norms with the token shift, beside one RMS norm that reads the stream and adds nothing
+        x, w1, w2, share = torch.randn(n, width, device=device), torch.ones(width, device=device), torch.ones(width, device=device), torch.rand(width, device=device)
+        states, sl = torch.zeros(8, width, device=device), i32(list(range(len(qs))))
+        us = timed(lambda: ops.shift_norm(x, w1, 1e-6, w2=w2, shift=share, states=states, ctx=ctx, state_slots=sl, out_dtype=bf))
+        hbm(f"shift_norm_{label}", us, n * width * 8 + 2 * len(qs) * width * 4, like="tenotar_rmsnorm (one norm)")
+        us = timed(lambda: ops.rmsnorm(x, w1, 1e-6, out_dtype=bf))
+        hbm(f"tenotar_rmsnorm_{label}", us, n * width * 6)
+        # the feed-forward's first product with gelu (decode: one kernel), beside the gated one with SwiGLU of as many weights
+        xb = torch.randn(n, width, device=device).to(bf)
+        up = (torch.randn(ff, width, device=device) * width ** -0.5).to(bf)
+        rows = torch.empty(n, B["heads"] * B["vdim"] + ff, device=device, dtype=bf)
+        into = rows[:, B["heads"] * B["vdim"] :]
+        us = timed(lambda: ops.linear_act(xb, up, "gelu", out=into))
+        work = (2.0 * n * width * ff) if prefill else (ff * width + n * (width + ff)) * 2
+        (tensor if prefill else hbm)(f"up_product_gelu_{label}", us, work, like="tenotar_gate_up_swiglu")
+        ff2 = twin["intermediate_size"]
+        gu, gb = (torch.randn(2 * ff2, width, device=device) * width ** -0.5).to(bf), torch.zeros(2 * ff2, device=device).to(bf)
+        us = timed(lambda: ops.swiglu(ops.linear(xb, gu), gb))
+        work = (4.0 * n * width * ff2) if prefill else (2 * ff2 * width + n * (width + ff2)) * 2
+        (tensor if prefill else hbm)(f"tenotar_gate_up_swiglu_{label}", us, work)
+        if prefill:
+            z = torch.randn(n, ff, device=device).to(bf)
+            us = timed(lambda: ops.unary(z, "gelu", out=into))
+            hbm(f"gelu_{label}", us, n * ff * 4, like="tenotar_swiglu")
+            z2 = torch.randn(n, 2 * ff2, device=device).to(bf)
+            us = timed(lambda: ops.swiglu(z2, gb))
+            hbm(f"tenotar_swiglu_{label}", us, n * ff2 * 6)
+        # the joined output product into the stream, beside the two products that a pre-norm layer runs
+        k1 = B["heads"] * B["vdim"]
+        wj = (torch.randn(width, k1 + ff, device=device) * (k1 + ff) ** -0.5).to(bf)
+        wo, wd = wj[:, :k1].contiguous(), wj[:, k1 : k1 + ff2].contiguous()
+        act = torch.randn(n, k1 + ff, device=device).to(bf)
+        sink = ops.ResidualSink(x, None, 0.0)
+        us = timed(lambda: sink.linear(act, wj))
+        work = (2.0 * n * width * (k1 + ff)) if prefill else ((k1 + ff) * width + n * (k1 + ff)) * 2 + n * width * 8
+        (tensor if prefill else hbm)(f"joined_output_product_{label}", us, work, like="tenotar_output_and_down_products")
+        a1, a2 = act[:, :k1].contiguous(), act[:, k1 : k1 + ff2].contiguous()
+        us = timed(lambda: (sink.linear(a1, wo), sink.linear(a2, wd)))
+        work = (2.0 * n * width * (k1 + ff2)) if prefill else ((k1 + ff2) * width + n * (k1 + ff2)) * 2 + n * width * 16
+        (tensor if prefill else hbm)(f"tenotar_output_and_down_products_{label}", us, work)
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -682,8 +781,8 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has (recorded in config)")
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64, the end-to-end run and the kernel table")
     ap.add_argument("--design", choices=["nurolorn-small", "nurolorn-1b", "kafepel-small", "kafepel-1b", "nudodra-small", "nudodra-1b", "tenotar-small",
-                                         "tenotar-1b"], default=None,
-                    help="instead of the one line: prefill and decode throughput of a Nurolorn, Kafepel, Nudodra or Tenotar configuration beside a Llama of "
+                                         "tenotar-1b", "pefedra-small", "pefedra-1b"], default=None,
+                    help="instead of the one line: prefill and decode throughput of a Nurolorn, Kafepel, Nudodra, Tenotar or Pefedra configuration beside a Llama of "
                          "equal width, depth and feed-forward size, and the design's own kernels against their rooflines")
     ap.add_argument("--sweep", action="store_true",
                     help="instead of the one line: a table of decode steps over batch sizes and context lengths and of prefills over prompt lengths")

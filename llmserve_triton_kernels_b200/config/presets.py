@@ -96,7 +96,24 @@ def _tenotar(width: int, pattern: str, heads: int, kv_heads: int, rank: int, q_r
     return {"architecture": "Tenotar", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6}, "logit_scale": 1.0}
 
 
+def _pefedra(width: int, pattern: str, heads: int, kv_heads: int, ff: int, span: int = 512, vocab: int = 32000) -> dict:
+    """``pattern``: one letter a layer, D attention with two score maps a head, T attention with rotated values.  Maps of 64 lanes;
+    a D head has two of them and values of 128 lanes (half as many heads), a T head values of 64; windows of ``span`` positions."""
+    head = 64
+    kinds = {
+        "D": lambda: {"type": "attention", "mixer": {"heads": heads // 2, "kv_heads": kv_heads // 2, "dim": head, "vdim": 2 * head, "scale": head ** -0.5,
+                                                     "diff": 0.5, "mask": {"size": span}, "rot": {"base": 10000.0, "dims": head, "scaling": {"factor": 4.0}}}},
+        "T": lambda: {"type": "attention_2", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5,
+                                                       "mask": {"size": span}, "rot": {"base": 10000.0, "dims": head // 2}}},
+    }
+    layers = [{**kinds[c](), "mlp": {"kind": "dense", "ff": ff}} for c in pattern]
+    return {"architecture": "Pefedra", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "layers": layers, "norm": {"eps": 1e-6}}
+
+
 PRESETS: dict[str, dict] = {
+    # Pefedra at the width and depth of the Tenotar presets below (the design has no published sizes)
+    "pefedra-small": _pefedra(1024, "DTTDTTDT", 16, 4, 4096),
+    "pefedra-1b": _pefedra(2048, "DTTDTTDTTDTT", 32, 8, 8192),
     # Tenotar at the sizes of the Nudodra and Kafepel presets below (the design has no published sizes)
     "tenotar-small": _tenotar(1024, "WCLWCLWC", 16, 4, 128, 384, 2816, 16, 2, 512, 1024),
     "tenotar-1b": _tenotar(2048, "WCLWCLWCLWCL", 32, 8, 256, 768, 5632, 32, 4, 704, 1408),

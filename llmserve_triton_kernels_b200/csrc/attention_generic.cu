@@ -160,7 +160,7 @@ LLM_EXPORT int llm_attention_rows(const void* q0, long long q0_token, long long 
         a.scale = scale; a.keep_first = keep_first; a.chunk = chunk; a.softcap = softcap;
         a.key_part = 0; a.keys1 = nullptr; a.k1_token = 0; a.fresh_d0 = 0; a.stats = nullptr;
         a.sinks = sinks; a.gate = gate; a.gate_token = gate_token; a.gate_per_head = gate_per_head;
-        a.maps = maps; a.q_map = q_map; a.k_map = k_map;
+        a.maps = maps; a.q_map = q_map; a.k_map = k_map; a.skip_from = 0;
         a.diff_weight = diff_weight; a.diff_eps = diff_eps; a.diff_scale = diff_scale;
         a.turn = (const float2*)turn; a.turn_neighbours = turn_neighbours;
     };

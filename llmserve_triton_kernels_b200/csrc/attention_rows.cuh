@@ -20,6 +20,7 @@ struct RowsArgs {
     const int *page_table, *token_request, *cu_tokens, *ctx_lens;
     const float* slopes;  // per query head: the score of key j for the query at position i loses slope * (i - j); null: none
     int table_width, n_tokens, H, KV, page_size, window;
+    int skip_from;  // > 0: requests that bring at least so many tokens are another kernel's
     // With a window, keys at positions below keep_first stay visible to every later query (0: none).  chunk > 0: a query
     // sees only keys of its own block of `chunk` positions, counted from position 0.
     int keep_first, chunk;

@@ -72,6 +72,7 @@ attention_rows_mma_kernel(const RowsArgs<bf16> a, int splits, float* __restrict_
     const int tile = (int)(gridDim.x / splits) - 1 - slot;
     const int group = a.H / a.KV;
     const int q_begin = a.cu_tokens[r], q_len = a.cu_tokens[r + 1] - q_begin, ctx_len = a.ctx_lens[r];
+    if (a.skip_from > 0 && q_len >= a.skip_from) return;
     const int rows_total = q_len * group, row0 = tile * TILE;
     if (row0 >= rows_total) return;
     const int first_pos = ctx_len - q_len;
@@ -397,6 +398,10 @@ attention_rows_merge_kernel(const RowsArgs<bf16> a, const float* __restrict__ pa
     pdl_wait();
     if (item >= (long long)a.n_tokens * a.H) return;
     const int t = (int)(item / a.H), h = (int)(item - (long long)t * a.H);
+    if (a.skip_from > 0) {
+        const int r = a.token_request[t];
+        if (a.cu_tokens[r + 1] - a.cu_tokens[r] >= a.skip_from) return;
+    }
     float y[8];
     for (int map = 0; map < a.maps; ++map) {
         const size_t first = ((size_t)item * a.maps + map) * splits;
@@ -529,7 +534,7 @@ int launch(const RowsArgs<bf16>& a, int requests, int max_query_len, int splits,
 }  // namespace
 
 // As llm_attention_rows, for bfloat16 with every run of lanes a multiple of 16 and 16-byte aligned rows; dv <= 256.
-// `max_query_len`: the most tokens a request brings (it sizes the grid).  `splits` > 1 cuts every row tile's keys over
+// `max_query_len`: the most tokens a request brings (it sizes the grid); skip_from > 0: requests of that many tokens and more are left out.  `splits` > 1 cuts every row tile's keys over
 // that many CTAs; part_o [n_tokens * H * maps * splits * dv] and part_ml [n_tokens * H * maps * splits * 2] (float32) then hold the
 // partial results until the merge that follows.  Returns LLM_ERR_UNSUPPORTED for shapes it does not take.
 LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long long q0_head, int d0, const void* q1,
@@ -543,7 +548,7 @@ LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long l
                                       long long k1_token, int fresh_d0, float* stats, const float* sinks, const float* gate,
                                       long long gate_token, int keep_first, int chunk, float softcap, int gate_per_head, int maps,
                                       long long q_map, long long k_map, float diff_weight, float diff_eps, float diff_scale,
-                                      const void* turn, int turn_neighbours, cudaStream_t stream) {
+                                      const void* turn, int turn_neighbours, int skip_from, cudaStream_t stream) {
     if (n_tokens <= 0 || requests <= 0) return 0;
     if (maps < 1 || maps > 2 || (maps == 2 && (d1 != 0 || sinks || key_part != 0 || stats)) || (turn && (key_part != 0 || stats)))
         return LLM_ERR_BAD_ARGUMENT;
@@ -579,7 +584,7 @@ LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long l
     a.key_part = key_part; a.keys1 = key_part == 2 ? (const bf16*)keys1 : nullptr; a.k1_token = k1_token; a.fresh_d0 = fresh_d0;
     a.stats = stats;
     a.sinks = sinks; a.gate = gate; a.gate_token = gate_token; a.gate_per_head = gate_per_head;
-    a.maps = maps; a.q_map = q_map; a.k_map = k_map;
+    a.maps = maps; a.q_map = q_map; a.k_map = k_map; a.skip_from = skip_from;
     a.diff_weight = diff_weight; a.diff_eps = diff_eps; a.diff_scale = diff_scale;
     a.turn = (const float2*)turn; a.turn_neighbours = turn_neighbours;
     const bool alias = key_part != 2 && values == keys && v_page == k_page && v_head == k_head && v_token == k_token;

@@ -40,7 +40,7 @@ using attn::AttnParams;
 constexpr int BM = 128, BN = 64, THREADS = 256, TMEM_COLS = 256;
 constexpr float LAZY = 8.f;  // log2 of how far a row's maximum may rise before its shift follows
 
-// What differs between the head sizes.  256 columns of tensor memory a CTA (two CTAs share an SM's 512), two
+// What differs between the sizes of a head: KD lanes of a query and a key, VD of a value.  256 columns of tensor memory a CTA (two CTAs share an SM's 512), two
 // bfloat16 to a column where an A operand lies:
 //   head size 64 : two tiles of scores [0, 64), [64, 128); the output [128, 192); the queries [192, 224); a tile's
 //                  probabilities [224, 256).  Three stages of keys and of values (16 KB a stage): 49 KB of shared memory.
@@ -48,13 +48,15 @@ constexpr float LAZY = 8.f;  // log2 of how far a row's maximum may rise before 
 //                  and stay in shared memory (32 KB, the first product's A operand from there); two stages of keys
 //                  and of values (32 KB a stage): 97 KB.  With one buffer of scores the product of tile j+1 starts when
 //                  the softmax has read tile j; the other CTA of the SM fills the gap.
-template <int HD>
+//   64 and 128   : one tile of scores [0, 64); the output [64, 192); the queries [192, 224); probabilities [224, 256).  Three stages
+//                  (24 KB): 73 KB.
+template <int KD, int VD>
 struct Shape {
-    static constexpr bool Q_IN_TMEM = HD == 64;
-    static constexpr int S_BUFFERS = HD == 64 ? 2 : 1, STAGES = HD == 64 ? 3 : 2;
-    static constexpr int O_COL = S_BUFFERS * BN, Q_COL = O_COL + HD, P_COL = Q_IN_TMEM ? Q_COL + HD / 2 : O_COL + HD;
-    static constexpr int HALVES = HD / 64;                // 64-wide pieces of a row of keys, values, queries: one TMA box each
-    static constexpr int K_BYTES = BN * HD * 2, STAGE_BYTES = 2 * K_BYTES, Q_BYTES = Q_IN_TMEM ? 0 : BM * HD * 2;
+    static constexpr bool Q_IN_TMEM = KD == 64;
+    static constexpr int S_BUFFERS = VD == 64 ? 2 : 1, STAGES = KD == 64 ? 3 : 2;
+    static constexpr int O_COL = S_BUFFERS * BN, Q_COL = O_COL + VD, P_COL = Q_IN_TMEM ? Q_COL + KD / 2 : O_COL + VD;
+    static constexpr int K_HALVES = KD / 64, V_HALVES = VD / 64;  // 64-wide pieces of a row of keys (queries), values: one TMA box each
+    static constexpr int K_BYTES = BN * KD * 2, V_BYTES = BN * VD * 2, STAGE_BYTES = K_BYTES + V_BYTES, Q_BYTES = Q_IN_TMEM ? 0 : BM * KD * 2;
     static constexpr size_t SMEM = 1024 + (size_t)Q_BYTES + (size_t)STAGES * STAGE_BYTES;
     static_assert(P_COL + BN / 2 <= TMEM_COLS, "tensor memory");
 };
@@ -64,18 +66,30 @@ struct TcParams {
     int min_tokens;         // requests with fewer tokens are other kernels'
     int tiles_per_request;  // 128-token tiles of the longest request
     int* error_flag;
+    // Heads of several score maps: blockIdx.x counts (head, map), the queries of a head's maps lie side by side, its keys' likewise
+    // in a row of the pool (map m from lane m * KD on), all maps over the same values.
+    int maps;
+    // The result of every (token, head, map) as it is, 32-bit [tokens, H * maps, VD], for a kernel that joins the maps; null: bfloat16 to a.out
+    float* raw;
+    // The values were cached turned by their positions' angles: lanes m and m + VD/2 of the result are turned back by the query
+    // token's row of (cos, sin) [tokens, VD / 2]; null: not
+    const float2* turn;
+    // One gate a head: the result times sigmoid(gate[token * gate_token + head]); null: none
+    const float* gate;
+    long long gate_token;
 };
 
 __device__ __forceinline__ void mbar_arrive(unsigned long long* bar) { tma::mbar_arrive(bar); }
 
-template <int HD>
+template <int KD, int VD>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kvmap) {
-    using Sh = Shape<HD>;
-    constexpr int STAGES = Sh::STAGES, NBUF = Sh::S_BUFFERS, K_BYTES = Sh::K_BYTES, STAGE_BYTES = Sh::STAGE_BYTES, HALVES = Sh::HALVES;
+    using Sh = Shape<KD, VD>;
+    constexpr int STAGES = Sh::STAGES, NBUF = Sh::S_BUFFERS, K_BYTES = Sh::K_BYTES, STAGE_BYTES = Sh::STAGE_BYTES;
+    constexpr int K_HALVES = Sh::K_HALVES, V_HALVES = Sh::V_HALVES;
     constexpr int O_COL = Sh::O_COL, Q_COL = Sh::Q_COL, P_COL = Sh::P_COL;
     const AttnParams& p = tp.a;
-    const int head = blockIdx.x, kvh = head / p.G;
+    const int q_head = blockIdx.x, head = q_head / tp.maps, kvh = head / p.G;
     const int r = blockIdx.y / tp.tiles_per_request;
     const int tile = tp.tiles_per_request - 1 - (int)(blockIdx.y % tp.tiles_per_request);  // long tiles first
     const int q_begin = p.cu_tokens[r], q_len = p.cu_tokens[r + 1] - q_begin;
@@ -94,7 +108,7 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     unsigned char* q_s = base;                // [halves][128 rows][64]: head size 128 only
-    unsigned char* kv_s = base + Sh::Q_BYTES;  // [STAGES][keys | values], each [halves][64 keys][64]
+    unsigned char* kv_s = base + Sh::Q_BYTES;  // [STAGES][keys | values], each [64-wide pieces][64 keys][64]
     __shared__ __align__(8) unsigned long long q_full, k_full[STAGES], k_empty[STAGES], v_full[STAGES], v_empty[STAGES], s_full[NBUF], s_empty[NBUF], p_full, o_full;
     __shared__ unsigned tmem_base;
     __shared__ int gave_up;
@@ -150,12 +164,13 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
         if (!Sh::Q_IN_TMEM && !is_v && lane == 0) {
             tma::mbar_expect_tx(&q_full, Sh::Q_BYTES);
 #pragma unroll
-            for (int h = 0; h < HALVES; ++h) tma::load_2d(q_s + (size_t)h * (BM * 128), &qmap, head * HD + h * 64, q_begin + row0, &q_full);
+            for (int h = 0; h < K_HALVES; ++h) tma::load_2d(q_s + (size_t)h * (BM * 128), &qmap, q_head * KD + h * 64, q_begin + row0, &q_full);
         }
         // One box per page and 64-wide piece, each issued by a lane of its own (a thread's TMA instructions follow one another slowly;
         // several threads' overlap).  The page table is read 32 entries at a time; a page outside the needed range is
         // replaced by one inside it.
-        const int first_page = t_begin * pages_per_tile;
+        const int first_page = t_begin * pages_per_tile, halves = is_v ? V_HALVES : K_HALVES;
+        const int lane0 = is_v ? 0 : (q_head - head * tp.maps) * KD;  // where a row's lanes of this map begin
         int my_page = 0, loaded_from = -32;
         bool alive = true;
         for (int j = 0; j < n_tiles && alive; ++j) {
@@ -169,15 +184,15 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
                     if (!gave_up) fail();
                     alive = false;
                 } else {
-                    tma::mbar_expect_tx(&full[s], K_BYTES);
+                    tma::mbar_expect_tx(&full[s], is_v ? Sh::V_BYTES : K_BYTES);
                 }
             }
             alive = __shfl_sync(0xffffffffu, (int)alive, 0) != 0;
-            const int in_tile = lane / HALVES, half = lane % HALVES;
+            const int in_tile = lane / halves, half = lane % halves;
             const int page = __shfl_sync(0xffffffffu, my_page, (idx0 - loaded_from + in_tile) & 31);
             if (alive && in_tile < pages_per_tile) {
                 unsigned char* dst = kv_s + (size_t)s * STAGE_BYTES + (size_t)is_v * K_BYTES + (size_t)half * (BN * 128) + (size_t)in_tile * ps * 128;
-                tma::load_2d(dst, &kvmap, half * 64, ((page * 2 + (int)is_v) * p.KV + kvh) * ps, &full[s]);
+                tma::load_2d(dst, &kvmap, lane0 + half * 64, ((page * 2 + (int)is_v) * p.KV + kvh) * ps, &full[s]);
             }
         }
     } else if (warp == 5) {
@@ -197,7 +212,7 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
                 asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
                 const unsigned char* k_tile = kv_s + (size_t)(j % STAGES) * STAGE_BYTES;
 #pragma unroll
-                for (int k = 0; k < HD / 16; ++k) {  // 16 of the head's lanes a step: piece k / 4 of the tile, 32 bytes further per step
+                for (int k = 0; k < KD / 16; ++k) {  // 16 of the head's lanes a step: piece k / 4 of the tile, 32 bytes further per step
                     const unsigned long long k_desc = umma::desc_sw128(k_tile + (size_t)(k / 4) * (BN * 128)) + 2 * (k % 4);
                     if constexpr (Sh::Q_IN_TMEM) {
                         umma::mma_bf16_ts(tmem_base + (j % NBUF) * BN, q_tmem + 8 * k, k_desc, IDESC_QK, k != 0);
@@ -214,7 +229,7 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
     } else if (warp == 7) {
         // ---- issuer of the second product: O += P_j V_j, as soon as the probabilities and the values are there ----
         if (lane == 0) {
-            constexpr unsigned IDESC_PV = umma::idesc_bf16(BM, HD, true);
+            constexpr unsigned IDESC_PV = umma::idesc_bf16(BM, VD, true);
             const unsigned o_tmem = tmem_base + O_COL, p_tmem = tmem_base + P_COL;
             bool ok = true;
             for (int j = 0; j < n_tiles && ok && !gave_up; ++j) {
@@ -224,7 +239,7 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
                 asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
                 // the values lie [key][d]: B with N contiguous; 16 keys are two atoms of 8 rows, 2048 bytes further per step
                 // (a head of 128 lanes is two such pieces side by side, BN * 128 bytes apart: the leading offset)
-                const unsigned long long v_desc = umma::desc_sw128(kv_s + (size_t)s * STAGE_BYTES + K_BYTES, (HALVES > 1 ? BN * 128 : 1024) >> 4);
+                const unsigned long long v_desc = umma::desc_sw128(kv_s + (size_t)s * STAGE_BYTES + K_BYTES, (V_HALVES > 1 ? BN * 128 : 1024) >> 4);
 #pragma unroll
                 for (int k = 0; k < BN / 16; ++k)  // the output accumulates over the tiles
                     umma::mma_bf16_ts(o_tmem, p_tmem + 8 * k, v_desc + (2048 >> 4) * k, IDESC_PV, k != 0 || j != 0);
@@ -245,9 +260,9 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
         const unsigned o_taddr = lane_base + O_COL;
         if constexpr (Sh::Q_IN_TMEM) {  // the row's queries, as they lie in memory (two to a word), into the row's lane of tensor memory
             unsigned qw[32];
-            const uint4* src = reinterpret_cast<const uint4*>(p.q + (size_t)(q_begin + tok) * p.q_stride + (size_t)head * HD);
+            const uint4* src = reinterpret_cast<const uint4*>(p.q + (size_t)(q_begin + tok) * p.q_stride + (size_t)q_head * KD);
 #pragma unroll
-            for (int c = 0; c < HD / 8; ++c) {
+            for (int c = 0; c < KD / 8; ++c) {
                 const uint4 u = row_ok ? src[c] : make_uint4(0, 0, 0, 0);
                 qw[4 * c] = u.x; qw[4 * c + 1] = u.y; qw[4 * c + 2] = u.z; qw[4 * c + 3] = u.w;
             }
@@ -342,7 +357,7 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
                 const float a = rescale ? alpha : 1.f;
                 const float2 a2 = make_float2(a, a);
 #pragma unroll 1
-                for (int h = 0; h < HALVES; ++h) {
+                for (int h = 0; h < V_HALVES; ++h) {
                     float o[64];
                     umma::tmem_ld64(o_taddr + 64 * h, o);
 #pragma unroll
@@ -372,13 +387,48 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
             if (lane == 0) fail();
         } else if (n_tiles > 0) {
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-            const float inv = 1.f / l_run;
-            __nv_bfloat16* dst = p.out + (size_t)(q_begin + tok) * p.out_stride + (size_t)head * HD;
+            float inv = 1.f / l_run;
+            __nv_bfloat16* dst = p.out + (size_t)(q_begin + tok) * p.out_stride + (size_t)head * VD;
+            if (tp.gate && row_ok) inv /= 1.f + expf(-tp.gate[(size_t)(q_begin + tok) * tp.gate_token + head]);
+            if (tp.turn) {
+                const float4* cs = reinterpret_cast<const float4*>(tp.turn + (size_t)(q_begin + tok) * (VD / 2));  // two pairs each
 #pragma unroll 1
-            for (int h = 0; h < HALVES; ++h) {
+                for (int h = 0; h < VD / 2; h += 32) {
+                    float a[32], b[32];
+                    umma::tmem_ld32(o_taddr + h, a);
+                    umma::tmem_ld32(o_taddr + VD / 2 + h, b);
+                    if (row_ok) {
+#pragma unroll
+                        for (int i = 0; i < 32; i += 2) {
+                            const float4 t = cs[(h + i) >> 1];
+                            const float u0 = a[i] * inv, v0 = b[i] * inv, u1 = a[i + 1] * inv, v1 = b[i + 1] * inv;
+                            a[i] = u0 * t.x + v0 * t.y;
+                            b[i] = v0 * t.x - u0 * t.y;
+                            a[i + 1] = u1 * t.z + v1 * t.w;
+                            b[i + 1] = v1 * t.z - u1 * t.w;
+                        }
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) {
+                            *reinterpret_cast<uint4*>(dst + h + c * 8) =
+                                make_uint4(attn::pack_bf16(a[c * 8], a[c * 8 + 1]), attn::pack_bf16(a[c * 8 + 2], a[c * 8 + 3]),
+                                           attn::pack_bf16(a[c * 8 + 4], a[c * 8 + 5]), attn::pack_bf16(a[c * 8 + 6], a[c * 8 + 7]));
+                            *reinterpret_cast<uint4*>(dst + VD / 2 + h + c * 8) =
+                                make_uint4(attn::pack_bf16(b[c * 8], b[c * 8 + 1]), attn::pack_bf16(b[c * 8 + 2], b[c * 8 + 3]),
+                                           attn::pack_bf16(b[c * 8 + 4], b[c * 8 + 5]), attn::pack_bf16(b[c * 8 + 6], b[c * 8 + 7]));
+                        }
+                    }
+                }
+            } else
+#pragma unroll 1
+            for (int h = 0; h < V_HALVES; ++h) {
                 float o[64];
                 umma::tmem_ld64(o_taddr + 64 * h, o);  // (by all lanes of the warp: the load is the warp's)
-                if (row_ok) {
+                if (row_ok && tp.raw) {
+                    float* raw = tp.raw + ((size_t)(q_begin + tok) * (p.H * tp.maps) + q_head) * VD + 64 * h;
+#pragma unroll
+                    for (int c = 0; c < 64; c += 4)
+                        *reinterpret_cast<float4*>(raw + c) = make_float4(o[c] * inv, o[c + 1] * inv, o[c + 2] * inv, o[c + 3] * inv);
+                } else if (row_ok) {
 #pragma unroll
                     for (int c = 0; c < 8; ++c) {
                         uint4 u;
@@ -408,43 +458,78 @@ attention_tcgen05_kernel(const TcParams tp, const __grid_constant__ CUtensorMap 
     }
 }
 
+// Two maps' results [tokens, H, 2, VD] (32-bit) become a head's: u = a1 - weight * a2, u / sqrt(mean(u^2) + eps) * scale, bfloat16.
+// A warp a (token, head); tokens of requests with fewer than min_tokens tokens are another kernel's.
+template <int VD>
+__global__ void __launch_bounds__(256)
+join_maps_kernel(const float* __restrict__ raw, const int* __restrict__ token_request, const int* __restrict__ cu_tokens, int min_tokens,
+                 int n_tokens, int H, float weight, float eps, float scale, __nv_bfloat16* __restrict__ out, long long out_token) {
+    constexpr int W = VD / 32;  // neighbouring lanes of a head a thread holds
+    pdl_trigger();
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (item >= (long long)n_tokens * H) return;
+    const int t = (int)(item / H), h = (int)(item - (long long)t * H), r = token_request[t];
+    if (cu_tokens[r + 1] - cu_tokens[r] < min_tokens) return;
+    pdl_wait();
+    const float* a = raw + (size_t)item * 2 * VD + lane * W;
+    float u[W], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < W; e += 2) {
+        const float2 x = *reinterpret_cast<const float2*>(a + e), y = *reinterpret_cast<const float2*>(a + VD + e);
+        u[e] = x.x - weight * y.x;
+        u[e + 1] = x.y - weight * y.y;
+        ss = fmaf(u[e], u[e], fmaf(u[e + 1], u[e + 1], ss));
+    }
+    const float norm = scale / sqrtf(warp_sum(ss) / (float)VD + eps);
+    __nv_bfloat16* o = out + (long long)t * out_token + (long long)h * VD + lane * W;
+#pragma unroll
+    for (int e = 0; e < W; e += 2) *reinterpret_cast<__nv_bfloat162*>(o + e) = __floats2bfloat162_rn(u[e] * norm, u[e + 1] * norm);
+}
+
 }  // namespace
 
 // The fewest tokens a request must bring for this kernel to take it (its CTAs are 128 tokens of one head).
 LLM_EXPORT int llm_attention_tcgen05_min_tokens() { return 128; }
 
 namespace {
-template <int HD>
-int launch_tcgen05(const TcParams& tp, const void* q, int q_stride, int n_tokens, const void* pool, long long kv_rows, int page_size,
-                   unsigned grid_y, cudaStream_t stream) {
-    using Sh = Shape<HD>;
+template <int KD, int VD>
+int launch_tcgen05(const TcParams& tp, const void* q, int q_stride, int n_tokens, const void* pool, long long kv_rows, int row_lanes,
+                   int page_size, unsigned grid_y, cudaStream_t stream) {
+    using Sh = Shape<KD, VD>;
     // one box of keys or values: a page's rows, 64 of the head's lanes; one box of queries: 128 tokens, 64 lanes of a head
-    const CUtensorMap* kvmap = tma::cached_map_2d_bf16(pool, (uint64_t)kv_rows, HD, HD, (uint32_t)page_size, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+    const CUtensorMap* kvmap = tma::cached_map_2d_bf16(pool, (uint64_t)kv_rows, (uint64_t)row_lanes, (uint64_t)row_lanes, (uint32_t)page_size, 64, CU_TENSOR_MAP_SWIZZLE_128B);
     const CUtensorMap* qmap = Sh::Q_IN_TMEM ? kvmap
-                                            : tma::cached_map_2d_bf16(q, (uint64_t)n_tokens, (uint64_t)tp.a.H * HD, (uint64_t)q_stride, BM, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+                                            : tma::cached_map_2d_bf16(q, (uint64_t)n_tokens, (uint64_t)tp.a.H * tp.maps * KD, (uint64_t)q_stride, BM, 64, CU_TENSOR_MAP_SWIZZLE_128B);
     if (!kvmap || !qmap) return LLM_ERR_UNSUPPORTED;
     static bool configured = false;  // per head size
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<KD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Sh::SMEM);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return launch_pdl(attention_tcgen05_kernel<HD>, dim3((unsigned)tp.a.H, grid_y), dim3(THREADS), Sh::SMEM, stream, tp, *qmap, *kvmap);
+    return launch_pdl(attention_tcgen05_kernel<KD, VD>, dim3((unsigned)(tp.a.H * tp.maps), grid_y), dim3(THREADS), Sh::SMEM, stream, tp, *qmap, *kvmap);
 }
-}  // namespace
 
-// Attention of the requests that bring at least min_tokens tokens (others are left untouched: another kernel's).
-// q: bfloat16 rows of q_stride elements that start with the H query heads; out: [tokens, H * D] with row stride
-// out_stride; pool: one layer's plane [pool_pages, 2, KV, page_size, D]; max_tokens: the most tokens of any request.
-// Takes head sizes 64 and 128, pages of 8, 16, 32 or 64 keys, 16-byte aligned rows; else LLM_ERR_UNSUPPORTED (nothing ran).
-LLM_EXPORT int llm_attention_tcgen05(const void* q, int q_stride, void* out, int out_stride, const void* pool, long long pool_pages,
-                                     const int* page_table, int table_width, const int* cu_tokens, const int* ctx_lens,
-                                     int requests, int n_tokens, int H, int KV, int D, int page_size, int window, float scale,
-                                     int min_tokens, int max_tokens, int* error_flag, cudaStream_t stream) {
+struct Differential {  // how two maps meet (raw == null: one map a head)
+    float* raw;
+    float weight, eps, scale;
+    const int* token_request;
+};
+
+int attention_tcgen05(const void* q, int q_stride, void* out, int out_stride, const void* pool, long long pool_pages, const int* page_table,
+                      int table_width, const int* cu_tokens, const int* ctx_lens, int requests, int n_tokens, int H, int KV, int KD, int VD,
+                      int row_lanes, int page_size, int window, float scale, int min_tokens, int max_tokens, const float2* turn, const float* gate,
+                      long long gate_token, const Differential& diff, int* error_flag, cudaStream_t stream) {
     if (n_tokens <= 0 || requests <= 0 || max_tokens < min_tokens) return 0;
-    if ((D != 64 && D != 128) || (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64)) return LLM_ERR_UNSUPPORTED;
-    if (H <= 0 || KV <= 0 || H % KV || table_width <= 0 || min_tokens < 1 || !(scale > 0.f)) return LLM_ERR_BAD_ARGUMENT;
-    if ((q_stride & 7) || (out_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) || ((uintptr_t)pool & 127) || q_stride < H * D)
+    const bool sizes = (KD == 64 && (VD == 64 || VD == 128)) || (KD == 128 && VD == 128);
+    if (!sizes || (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64)) return LLM_ERR_UNSUPPORTED;
+    const int maps = diff.raw ? 2 : 1;
+    if (H <= 0 || KV <= 0 || H % KV || table_width <= 0 || min_tokens < 1 || !(scale > 0.f) || row_lanes < maps * KD || row_lanes < VD ||
+        (diff.raw && (turn || gate || !diff.token_request)))
+        return LLM_ERR_BAD_ARGUMENT;
+    if ((q_stride & 7) || (out_stride & 7) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) || ((uintptr_t)pool & 127) || q_stride < H * maps * KD ||
+        (row_lanes & 7) || ((uintptr_t)turn & 15) || ((uintptr_t)diff.raw & 15))
         return LLM_ERR_UNSUPPORTED;
     const long long kv_rows = pool_pages * 2 * KV * page_size;
     if (kv_rows <= 0 || kv_rows > 0x7fffffffLL) return LLM_ERR_UNSUPPORTED;
@@ -466,8 +551,50 @@ LLM_EXPORT int llm_attention_tcgen05(const void* q, int q_stride, void* out, int
     tp.min_tokens = min_tokens;
     tp.tiles_per_request = (max_tokens + BM - 1) / BM;
     tp.error_flag = error_flag;
+    tp.maps = maps;
+    tp.raw = diff.raw;
+    tp.turn = turn;
+    tp.gate = gate;
+    tp.gate_token = gate_token;
     const long long y = (long long)requests * tp.tiles_per_request;
     if (y > 65535) return LLM_ERR_UNSUPPORTED;
-    return D == 64 ? launch_tcgen05<64>(tp, q, q_stride, n_tokens, pool, kv_rows, page_size, (unsigned)y, stream)
-                   : launch_tcgen05<128>(tp, q, q_stride, n_tokens, pool, kv_rows, page_size, (unsigned)y, stream);
+    int code;
+    if (KD == 64 && VD == 64) code = launch_tcgen05<64, 64>(tp, q, q_stride, n_tokens, pool, kv_rows, row_lanes, page_size, (unsigned)y, stream);
+    else if (KD == 64) code = launch_tcgen05<64, 128>(tp, q, q_stride, n_tokens, pool, kv_rows, row_lanes, page_size, (unsigned)y, stream);
+    else code = launch_tcgen05<128, 128>(tp, q, q_stride, n_tokens, pool, kv_rows, row_lanes, page_size, (unsigned)y, stream);
+    if (code != 0 || maps == 1) return code;
+    const long long items = (long long)n_tokens * H;
+    auto join = [&](auto kernel) {
+        return launch_pdl(kernel, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream, (const float*)diff.raw, diff.token_request, cu_tokens, min_tokens,
+                          n_tokens, H, diff.weight, diff.eps, diff.scale, (__nv_bfloat16*)out, (long long)out_stride);
+    };
+    return VD == 64 ? join(join_maps_kernel<64>) : join(join_maps_kernel<128>);
+}
+}  // namespace
+
+// Attention of the requests that bring at least min_tokens tokens (others are left untouched: another kernel's).
+// q: bfloat16 rows of q_stride elements that start with the H query heads; out: [tokens, H * D] with row stride
+// out_stride; pool: one layer's plane [pool_pages, 2, KV, page_size, D]; max_tokens: the most tokens of any request.
+// Takes head sizes 64 and 128, pages of 8, 16, 32 or 64 keys, 16-byte aligned rows; else LLM_ERR_UNSUPPORTED (nothing ran).
+LLM_EXPORT int llm_attention_tcgen05(const void* q, int q_stride, void* out, int out_stride, const void* pool, long long pool_pages,
+                                     const int* page_table, int table_width, const int* cu_tokens, const int* ctx_lens,
+                                     int requests, int n_tokens, int H, int KV, int D, int page_size, int window, float scale,
+                                     int min_tokens, int max_tokens, int* error_flag, cudaStream_t stream) {
+    return attention_tcgen05(q, q_stride, out, out_stride, pool, pool_pages, page_table, table_width, cu_tokens, ctx_lens, requests, n_tokens, H, KV, D, D,
+                             D, page_size, window, scale, min_tokens, max_tokens, nullptr, nullptr, 0, Differential{}, error_flag, stream);
+}
+
+// The same with keys of KD and values of VD lanes (64 and 64, 64 and 128, 128 and 128) in rows of row_lanes; `turn` [tokens, VD / 2] pairs
+// (cos, sin) or null: values that turn back; `gate` (row pitch gate_token) or null: one gate a head; `raw` [tokens, H, 2, VD] (32-bit
+// scratch) or null: two score maps a head, whose results meet as u / sqrt(mean(u^2) + diff_eps) * diff_scale, u = a1 - diff_weight * a2
+// (a second launch; without turn and gate).
+LLM_EXPORT int llm_attention_tcgen05_general(const void* q, int q_stride, void* out, int out_stride, const void* pool, long long pool_pages,
+                                             const int* page_table, int table_width, const int* token_request, const int* cu_tokens,
+                                             const int* ctx_lens, int requests, int n_tokens, int H, int KV, int KD, int VD, int row_lanes,
+                                             int page_size, int window, float scale, int min_tokens, int max_tokens, const void* turn,
+                                             const float* gate, long long gate_token, float* raw, float diff_weight, float diff_eps,
+                                             float diff_scale, int* error_flag, cudaStream_t stream) {
+    const Differential diff = {raw, diff_weight, diff_eps, diff_scale, token_request};
+    return attention_tcgen05(q, q_stride, out, out_stride, pool, pool_pages, page_table, table_width, cu_tokens, ctx_lens, requests, n_tokens, H, KV, KD, VD,
+                             row_lanes, page_size, window, scale, min_tokens, max_tokens, (const float2*)turn, gate, gate_token, diff, error_flag, stream);
 }

@@ -16,7 +16,8 @@
 //   warm:      queries times 1 + coef * ln(floor((position + 1) / every) + 1)
 // Queries go to q_out [N, Hq * D]; keys and values into the token's slot of pool [pages, 2, Hk, page_size, Dp].  With maps = 2
 // every two key heads in a row share a value head and a row of the pool [pages, 2, Hk / 2, page_size, Dp], side by side.
-// Everything is computed in 32-bit.  One CTA per token, one warp per head at a time.
+// Everything is computed in 32-bit.  One CTA per token, one warp per head at a time; where no head is normed by itself and
+// everything lies on boundaries of four lanes, a second kernel takes four neighbouring pairs of lanes a thread instead.
 #include <type_traits>
 
 #include "common.cuh"
@@ -149,6 +150,102 @@ head_prepare_kernel(const TI* __restrict__ proj, int ldp, const float* __restric
     }
 }
 
+// No norm, or one over whole projections; half layout; no factor on the queries, no values kept or mixed; D, rot / 2, V (and V / 2
+// where the values turn), the pitches and Dp multiples of four.  A thread takes four neighbouring pairs of a head, or four lanes
+// that pass, at a time (16-byte loads, 8- or 16-byte stores).  Grid (tokens, shares): a token's items may be shared out over several
+// CTAs (steps of few tokens), each of which works out the token's angles and sums for itself.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+head_prepare_wide_kernel(const float* __restrict__ proj, int ldp, const float* __restrict__ bias, TO* __restrict__ q_out, int ldq,
+                         TO* __restrict__ pool, const int* __restrict__ slot_map, int page_size, int Dp, const float* __restrict__ qw,
+                         const float* __restrict__ kw, float eps, const float* __restrict__ freq, int rot, const int* __restrict__ positions,
+                         int Hq, int Hk, int D, int V, int maps, const float* __restrict__ v_freq, float2* __restrict__ turn_out) {
+    extern __shared__ float2 turn[];  // rot / 2 (cos, sin), then V / 2 for the values
+    __shared__ float scratch[33];
+    pdl_trigger();
+    const int t = blockIdx.x, half = rot >> 1, v_half = v_freq ? V >> 1 : 0, Gv = Hk / maps;
+    const float position = half + v_half > 0 ? (float)positions[t] : 0.f;
+    for (int i = threadIdx.x; i < half + v_half; i += blockDim.x) {
+        float s, c;
+        sincosf(position * (i < half ? freq[i] : v_freq[i - half]), &s, &c);
+        turn[i] = make_float2(c, s);
+    }
+    const int slot = Hk > 0 ? slot_map[t] : 0;
+    const int page = slot / page_size, off = slot - page * page_size;
+    __syncthreads();
+    pdl_wait();
+    if (turn_out && blockIdx.y == 0)
+        for (int i = threadIdx.x; i < v_half; i += blockDim.x) turn_out[(size_t)t * v_half + i] = turn[half + i];
+    const float* row = proj + (size_t)t * ldp;
+    auto load = [&](int c, float (&v)[4]) {
+        load4(row + c, v);
+        if (bias) {
+            float b[4];
+            load4(bias + c, b);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] += b[e];
+        }
+    };
+    float whole[2] = {1.f, 1.f};
+    if (qw) {
+        float sums[2] = {0.f, 0.f};
+        for (int c = threadIdx.x * 4; c < (Hq + Hk) * D; c += blockDim.x * 4) {
+            float v[4];
+            load(c, v);
+            const float s = fmaf(v[0], v[0], v[1] * v[1]) + fmaf(v[2], v[2], v[3] * v[3]);
+            if (c < Hq * D) sums[0] += s;
+            else sums[1] += s;
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) whole[e] = 1.f / sqrtf(block_sum(sums[e], scratch) / (float)((e ? Hk : Hq) * D) + eps);
+    }
+    const int pairs = half >> 2, per = pairs + ((D - rot) >> 2), per_v = v_half > 0 ? v_half >> 2 : V >> 2;
+    const int heads_items = (Hq + Hk) * per, items = heads_items + Gv * per_v;
+    for (int it = blockIdx.y * blockDim.x + threadIdx.x; it < items; it += gridDim.y * blockDim.x) {
+        const bool is_v = it >= heads_items;
+        const int local = is_v ? it - heads_items : it, span = is_v ? per_v : per;
+        const int head = local / span, i = local - head * span;
+        const bool turns = is_v ? v_half > 0 : i < pairs;
+        const int da = turns ? 4 * i : is_v ? 4 * i : 4 * i + half;  // (lanes that pass follow the rotated ones: rot + 4 (i - pairs))
+        const int src = is_v ? (Hq + Hk) * D + head * V : head * D;
+        float a[4], b[4];
+        load(src + da, a);
+        if (turns) load(src + da + (is_v ? v_half : half), b);
+        if (!is_v && qw) {
+            const bool is_q = head < Hq;
+            const float* w = is_q ? qw + head * D : kw + (head - Hq) * D;
+            const float s = whole[is_q ? 0 : 1];
+            float x[4];
+            load4(w + da, x);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[e] = a[e] * s * x[e];
+            if (turns) {
+                load4(w + da + half, x);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) b[e] = b[e] * s * x[e];
+            }
+        }
+        TO* dst;
+        if (is_v) dst = pool + ((((size_t)page * 2 + 1) * Gv + head) * page_size + off) * Dp;
+        else if (head < Hq) dst = q_out + (size_t)t * ldq + head * D;
+        else {
+            const int k = head - Hq, kh = k / maps;
+            dst = pool + (((size_t)page * 2 * Gv + kh) * page_size + off) * Dp + (k - kh * maps) * D;
+        }
+        if (turns) {
+            const float2* cs = turn + (is_v ? half : 0) + 4 * i;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float u = a[e], v = b[e];
+                a[e] = u * cs[e].x - v * cs[e].y;
+                b[e] = v * cs[e].x + u * cs[e].y;
+            }
+            store4(dst + da + (is_v ? v_half : half), b);
+        }
+        store4(dst + da, a);
+    }
+}
+
 }  // namespace
 
 // in_dtype: the projections' type; out_dtype: the type of the queries on their way out and of the pool.
@@ -166,6 +263,23 @@ LLM_EXPORT int llm_head_prepare(const void* proj, int in_dtype, int ldp, const f
         (normed && (!qw || (Hk > 0 && !kw))) || (Hq > 0 && !q_out) || ((v_keep || v_first) && (values_are_keys || Hk <= 0)))
         return LLM_ERR_BAD_ARGUMENT;
     using bf = __nv_bfloat16;
+    auto aligned = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const int v_lanes = v_freq ? V / 2 : V;
+    if (in_dtype == LLM_F32 && normed != 1 && !interleaved && !values_are_keys && warm_every <= 0 && !v_keep && !v_first &&
+        ((D | (rot / 2) | (Hk > 0 ? v_lanes | Dp : 0) | ldp | ldq) & 3) == 0 && aligned(proj) && aligned(bias) && aligned(q_out) && aligned(pool) &&
+        aligned(qw) && aligned(kw)) {
+        const int items = (Hq + Hk) * (D / 4 - rot / 8) + (Hk / maps) * (v_lanes / 4);
+        int shares = (2 * 148 + N - 1) / N, most = (items + 255) / 256;
+        if (shares > most) shares = most;
+        const size_t wide_smem = (size_t)(rot / 2 + (v_freq ? V / 2 : 0) + 1) * sizeof(float2);
+        auto wide = [&](auto kernel, auto* qo) {
+            using TO = std::remove_pointer_t<decltype(qo)>;
+            return launch_pdl(kernel, dim3(N, shares < 1 ? 1 : shares), dim3(256), wide_smem, stream, (const float*)proj, ldp, bias, qo, ldq, (TO*)pool,
+                              slot_map, page_size, Dp, normed ? qw : nullptr, kw, eps, freq, rot, positions, Hq, Hk, D, V, maps, v_freq, (float2*)turn_out);
+        };
+        if (out_dtype == LLM_F32) return wide(head_prepare_wide_kernel<float>, (float*)q_out);
+        if (out_dtype == LLM_BF16) return wide(head_prepare_wide_kernel<bf>, (bf*)q_out);
+    }
     const size_t smem = ((size_t)WARPS * D + 1) * sizeof(float) + (size_t)(rot / 2 + 1 + (v_freq ? V / 2 : 0)) * sizeof(float2);
     auto go = [&](auto kernel, auto* in, auto* qo) {
         using TK = std::remove_pointer_t<decltype(qo)>;

@@ -188,26 +188,69 @@ __device__ __forceinline__ float unary_of(float v, int kind, float alpha) {
 
 template <typename T>
 __global__ void unary_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int ldo, int cols, size_t total,
-                             int kind, float alpha, bool wide) {
+                             int kind, float alpha) {
     pdl_trigger();
     pdl_wait();
     const size_t stride = (size_t)gridDim.x * blockDim.x;
-    if (wide) {  // four elements a thread: rows a multiple of four long and apart, bases aligned
-        for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < total; i += stride * 4) {
-            const size_t t = i / cols;
-            const int j = (int)(i - t * cols);
-            float v[4];
-            load4(x + t * ldx + j, v);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) v[e] = unary_of(v[e], kind, alpha);
-            store4(out + t * ldo + j, v);
-        }
-        return;
-    }
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
         const size_t t = i / cols;
         const int j = (int)(i - t * cols);
         out[t * ldo + j] = from_float<T>(unary_of(to_float(x[t * ldx + j]), kind, alpha));
+    }
+}
+
+// The same with eight elements a thread (rows and pitches multiples of eight, bases aligned): grid (pieces of a row, rows).
+template <typename T, int KIND>
+__global__ void __launch_bounds__(256) unary_wide_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int ldo, int rows, int cols, float alpha) {
+    pdl_trigger();
+    const int j = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    pdl_wait();
+    if (j >= cols) return;
+    for (int t = blockIdx.y; t < rows; t += gridDim.y) {
+        float v[8];
+        float (&lo)[4] = reinterpret_cast<float (&)[4]>(v[0]);
+        float (&hi)[4] = reinterpret_cast<float (&)[4]>(v[4]);
+        if constexpr (sizeof(T) == 2) {
+            const uint4 u = *reinterpret_cast<const uint4*>(x + (size_t)t * ldx + j);
+            const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const __nv_bfloat162 b = *reinterpret_cast<const __nv_bfloat162*>(&w[e]);
+                v[2 * e] = __low2float(b);
+                v[2 * e + 1] = __high2float(b);
+            }
+        } else {
+            load4(x + (size_t)t * ldx + j, lo);
+            load4(x + (size_t)t * ldx + j + 4, hi);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = unary_of(v[e], KIND, alpha);
+        if constexpr (sizeof(T) == 2) {
+            unsigned w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+                w[e] = *reinterpret_cast<const unsigned*>(&b);
+            }
+            *reinterpret_cast<uint4*>(out + (size_t)t * ldo + j) = make_uint4(w[0], w[1], w[2], w[3]);
+        } else {
+            store4(out + (size_t)t * ldo + j, lo);
+            store4(out + (size_t)t * ldo + j + 4, hi);
+        }
+    }
+}
+
+template <typename T>
+int unary_wide(const T* x, int ldx, T* out, int ldo, int rows, int cols, int kind, float alpha, cudaStream_t stream) {
+    const int pieces = cols / 8, threads = pieces >= 256 ? 256 : (pieces + 31) / 32 * 32;
+    const dim3 grid((pieces + threads - 1) / threads, rows < 65535 ? rows : 65535);
+    auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(threads), 0, stream, x, ldx, out, ldo, rows, cols, alpha); };
+    switch (kind) {
+        case 0: return go(unary_wide_kernel<T, 0>);
+        case 1: return go(unary_wide_kernel<T, 1>);
+        case 2: return go(unary_wide_kernel<T, 2>);
+        case 3: return go(unary_wide_kernel<T, 3>);
+        default: return go(unary_wide_kernel<T, 4>);
     }
 }
 
@@ -303,14 +346,17 @@ LLM_EXPORT int llm_unary(const void* x, int ldx, void* out, int ldo, int dtype, 
     if (rows <= 0 || cols <= 0) return 0;
     if (ldx < cols || ldo < cols || kind < 0 || kind > 4) return LLM_ERR_BAD_ARGUMENT;
     const size_t total = (size_t)rows * cols;
-    const bool wide = ((cols | ldx | ldo) & 3) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0;
-    const int threads = 256, blocks = flat_blocks(wide ? (total + 3) / 4 : total, threads);
+    if (((cols | ldx | ldo) & 7) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0) {
+        if (dtype == LLM_F32) return unary_wide<float>((const float*)x, ldx, (float*)out, ldo, rows, cols, kind, alpha, stream);
+        if (dtype == LLM_BF16) return unary_wide<__nv_bfloat16>((const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, rows, cols, kind, alpha, stream);
+    }
+    const int threads = 256, blocks = flat_blocks(total, threads);
     if (dtype == LLM_F32)
         return launch_pdl(unary_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float*)x, ldx, (float*)out, ldo,
-                          cols, total, kind, alpha, wide);
+                          cols, total, kind, alpha);
     if (dtype == LLM_BF16)
         return launch_pdl(unary_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16*)x, ldx,
-                          (__nv_bfloat16*)out, ldo, cols, total, kind, alpha, wide);
+                          (__nv_bfloat16*)out, ldo, cols, total, kind, alpha);
     return LLM_ERR_BAD_ARGUMENT;
 }
 

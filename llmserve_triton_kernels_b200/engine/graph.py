@@ -18,6 +18,8 @@ time, and what one keeps between replays (its logits) is never freed.
 
 from __future__ import annotations
 
+import gc
+
 import numpy as np
 import torch
 
@@ -133,8 +135,16 @@ class StepGraph:
         graph = torch.cuda.CUDAGraph()
         before = ops.launch_count()
         pool = getattr(self.owner, "graph_pool", None)
-        with torch.cuda.graph(graph, pool=pool):
-            self.logits = self.model.forward(self.ctx, self.views)
+        # a garbage collection in the middle of the capture may destroy graphs of a step function that is gone (it and its
+        # graphs refer to one another), which CUDA does not permit while a stream is being captured
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(graph, pool=pool):
+                self.logits = self.model.forward(self.ctx, self.views)
+        finally:
+            if collecting:
+                gc.enable()
         if self.owner is not None and pool is None:
             self.owner.graph_pool = graph.pool()
         self.launches = ops.launch_count() - before

@@ -56,7 +56,9 @@ _SIGNATURES = {
                            _i, _i, _ll, _ll, _f, _f, _f, _vp, _i, _vp],
     "llm_attention_rows_mma": [_vp, _ll, _ll, _i, _vp, _ll, _ll, _i, _vp, _ll, _ll, _vp, _ll, _ll, _ll, _vp, _ll, _ll, _ll, _i,
                                _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp, _ll, _i, _vp, _vp, _vp, _ll, _i, _i, _f,
-                               _i, _i, _ll, _ll, _f, _f, _f, _vp, _i, _vp],
+                               _i, _i, _ll, _ll, _f, _f, _f, _vp, _i, _i, _vp],
+    "llm_attention_tcgen05_general": [_vp, _i, _vp, _i, _vp, _ll, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _vp,
+                                      _vp, _ll, _vp, _f, _f, _f, _vp, _vp],
     "llm_gemm_simt_batched": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _ll, _ll, _ll, _vp],
     "llm_sample": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
     "llm_sigmoid_attention": [_vp, _i, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i,
@@ -1098,13 +1100,19 @@ def head_linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return torch.bmm(x.transpose(0, 1), w.transpose(1, 2)).transpose(0, 1)
 
 
+# Keys that one of several CTAs on a tile of rows takes at least; an SM gets two such CTAs (one where values are longer than 128
+# lanes: no second one fits).  Measured with the merge behind it, against 256 keys and one CTA an SM: 32 heads on 8 of 64 lanes, window
+# 512: 18.4 -> 12.4 us for one request, 22.1 -> 14.1 us for 8; all of 2,048 keys, 8 requests: 73.0 -> 38.9 us.
+_ROWS_SPLIT_KEYS = 128
+
+
 def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, page_table, page_size: int, ctx, *, num_heads: int,
                    num_kv_heads: int, scale: float, window: int | None = None, slopes: torch.Tensor | None = None,
                    key_part: int = 0, keys1: int | None = None, k1_token: int = 0, fresh_d0: int = 0, want_stats: bool = False,
                    leave_parts: bool = False, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
                    keep_first: int | None = None, chunk: int | None = None, softcap: float | None = None, gate_per_head: bool = False,
                    differential: "DifferentialMaps | None" = None, turn: torch.Tensor | None = None, turn_neighbours: bool = False,
-                   out: torch.Tensor | None = None):
+                   out: torch.Tensor | None = None, skip_from: int = 0):
     """Attention in its general form: queries ``q0 [N, H, d0]`` and optionally ``q1 [N, H, d1]`` (lanes behind q0's),
     keys and values addressed by ``(page, head, token)`` strides in elements, an optional bias ``-slopes[h] * distance``.
     Returns ``[N, H, value_dim]``.
@@ -1124,7 +1132,8 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
     each has a softmax over the same values and the head's output is the norm of their difference.  ``turn`` (float32
     ``[N, value_dim / 2, 2]``, cosines and sines): pair m of a head's output, lanes m and m + value_dim/2 (``turn_neighbours``:
     2m and 2m + 1), is turned back by the token's angle (the values were cached turned by theirs).  ``out``: where the result
-    goes, ``[N, H, value_dim]`` with any token stride."""
+    goes, ``[N, H, value_dim]`` with any token stride.  ``skip_from``: requests that bring at least so many tokens may be left out
+    (another kernel has them)."""
     maps = 2 if differential is not None else 1
     n, d0 = q0.shape[0], q0.shape[2] // maps
     _need(q0.shape[2] == maps * d0, "attention_rows: two maps a head have queries of an even number of lanes")
@@ -1154,12 +1163,13 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
         # the tensor cores: 64 rows of (token, group member) a CTA; few CTAs and long contexts: the keys cut over several
         group = num_heads // num_kv_heads
         longest = getattr(ctx, "max_context_len", None) or int(ctx.context_lens.max())
+        most = _most_tokens_below(ctx, skip_from) if skip_from else ctx.max_query_len
         if window:
-            longest = min(longest, window + keep_first + ctx.max_query_len)
+            longest = min(longest, window + keep_first + most)
         if chunk:
-            longest = min(longest, chunk + ctx.max_query_len)
-        ctas = -(-ctx.max_query_len * group * maps // 64) * num_kv_heads * ctx.num_requests
-        splits = max(1, min(-(-longest // 256), _sm_count() // ctas, 16, _SPLIT_SCRATCH_BYTES // (n * num_heads * maps * value_dim * 4)))
+            longest = min(longest, chunk + most)
+        ctas = -(-most * group * maps // 64) * num_kv_heads * ctx.num_requests
+        splits = max(1, min(-(-longest // _ROWS_SPLIT_KEYS), (2 if value_dim <= 128 else 1) * _sm_count() // ctas, 16, _SPLIT_SCRATCH_BYTES // (n * num_heads * maps * value_dim * 4)))
         if key_part or want_stats:
             splits = 1
         stats = torch.empty((n, num_heads, 2), dtype=torch.float32, device=q0.device) if want_stats else None
@@ -1172,9 +1182,9 @@ def attention_rows(q0, q1, keys, k_strides, values, v_strides, value_dim: int, p
             0 if q1 is None else q1.stride(1), d1, None if (leave_parts and splits > 1) else _ptr(out), out.stride(0), out.stride(1),
             keys, *k_strides, values, *v_strides,
             value_dim, _ptr(page_table), page_table.shape[1], _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.context_lens),
-            _ptr(slopes), n, ctx.num_requests, ctx.max_query_len, num_heads, num_kv_heads, page_size, int(window or 0), float(scale),
+            _ptr(slopes), n, ctx.num_requests, most, num_heads, num_kv_heads, page_size, int(window or 0), float(scale),
             splits, _ptr(part_o), _ptr(part_ml), int(key_part), keys1, int(k1_token), int(fresh_d0), _ptr(stats), _ptr(sinks), _ptr(gate),
-            gate_token, keep_first, chunk, softcap, *more, _stream(),
+            gate_token, keep_first, chunk, softcap, *more, int(skip_from), _stream(),
         )
         if code != 10002:
             _check(code, "attention_rows (tensor cores)")
@@ -1322,12 +1332,68 @@ def paged_softmax_attention(q: torch.Tensor, pool: torch.Tensor, page_table: tor
     if out is not None:
         _need(out.dim() == 2 and tuple(out.shape) == (q.shape[0], num_heads * value_dim) and out.stride(1) == 1 and out.dtype == q.dtype,
               "paged_softmax_attention: out [N, heads * value_dim] of the queries' type")
-    o3 = None if out is None else out.as_strided((q.shape[0], num_heads, value_dim), (out.stride(0), value_dim, 1), out.storage_offset())
-    done = attention_rows(q3, None, _ptr(pool), (page, head, row), values, (page, head, row), value_dim, page_table, page_size, ctx,
-                          num_heads=num_heads, num_kv_heads=num_kv_heads, scale=scale, window=window, sinks=sinks, gate=gate,
-                          keep_first=keep_first, chunk=chunk, softcap=softcap, slopes=slopes, gate_per_head=gate_per_head,
-                          differential=differential, turn=turn, turn_neighbours=turn_neighbours, out=o3)
-    return done.view(q.shape[0], num_heads * value_dim) if out is None else out
+    if out is None:
+        out = torch.empty((q.shape[0], num_heads * value_dim), dtype=q.dtype, device=q.device)
+    taken = 0  # requests of at least so many tokens that the tcgen05 kernel has taken
+    if sinks is None and not keep_first and not chunk and not softcap and slopes is None and not turn_neighbours and (gate is None or gate_per_head):
+        taken, rest = _tcgen05_softmax_attention(q, pool, page_table, ctx, out, num_heads, num_kv_heads, key_dim // (2 if differential is not None else 1),
+                                                 value_dim, scale, window, gate, differential, turn)
+        if taken and not rest:
+            return out
+    o3 = out.as_strided((q.shape[0], num_heads, value_dim), (out.stride(0), value_dim, 1), out.storage_offset())
+    attention_rows(q3, None, _ptr(pool), (page, head, row), values, (page, head, row), value_dim, page_table, page_size, ctx,
+                   num_heads=num_heads, num_kv_heads=num_kv_heads, scale=scale, window=window, sinks=sinks, gate=gate,
+                   keep_first=keep_first, chunk=chunk, softcap=softcap, slopes=slopes, gate_per_head=gate_per_head,
+                   differential=differential, turn=turn, turn_neighbours=turn_neighbours, out=o3, skip_from=taken)
+    return out
+
+
+def _token_counts(ctx) -> list[int]:
+    cu = getattr(ctx, "host_cu_tokens", None)
+    if cu is None:
+        cu = ctx.cu_tokens.tolist()
+    return [b - a for a, b in zip(cu, cu[1:])]
+
+
+def _most_tokens_below(ctx, limit: int) -> int:
+    """The most tokens that a request with fewer than ``limit`` tokens brings."""
+    return max((c for c in _token_counts(ctx) if c < limit), default=1)
+
+
+_TC_SOFTMAX_SIZES = ((64, 64), (64, 128), (128, 128))  # lanes of a key (of one map) and of a value
+
+
+def _tcgen05_softmax_attention(q, pool, page_table, ctx, out, heads: int, kv_heads: int, key_dim: int, value_dim: int, scale: float,
+                               window, gate, differential, turn) -> tuple[int, bool]:
+    """The part of :func:`paged_softmax_attention` that the tcgen05 kernel takes: bfloat16 requests that bring at least
+    ``_TC_ATTENTION_MIN_TOKENS`` tokens.  Returns ``(that number or 0 if it took none, whether other requests are left)``."""
+    if (q.dtype != torch.bfloat16 or _FORCE_GENERIC_ATTENTION or not _TC_ATTENTION_ENABLED or (key_dim, value_dim) not in _TC_SOFTMAX_SIZES
+            or pool.shape[3] not in _TC_ATTENTION_PAGE_SIZES or (differential is not None and (gate is not None or turn is not None))
+            or ctx.max_query_len < _TC_ATTENTION_MIN_TOKENS):
+        return 0, True
+    if turn is not None:
+        _need(turn.dtype == torch.float32 and turn.is_contiguous() and tuple(turn.shape) == (q.shape[0], value_dim // 2, 2), "turn: float32 [N, value_dim / 2, 2]")
+    if gate is not None:
+        _need(gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape[0] == q.shape[0] and gate.shape[1] >= heads, "the gate must be float32 [N, heads]")
+    _i32(page_table, "page_table")
+    counts = _token_counts(ctx)
+    n = q.shape[0]
+    raw = None
+    if differential is not None:
+        raw = torch.empty((n, heads, 2, value_dim), dtype=torch.float32, device=q.device)
+    weight, eps, post = (differential.weight, differential.eps, differential.scale) if differential is not None else (0.0, 0.0, 0.0)
+    code = _launch(
+        "llm_attention_tcgen05_general", _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(pool), pool.shape[0], _ptr(page_table), page_table.shape[1],
+        _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.context_lens), len(counts), n, heads, kv_heads, key_dim, value_dim, pool.shape[4], pool.shape[3],
+        int(window or 0), float(scale), _TC_ATTENTION_MIN_TOKENS, max(counts), _ptr(turn), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(raw),
+        float(weight), float(eps), float(post), _error_flag_ptr(), _stream(),
+    )
+    if code == 10002:
+        add_launches(-1)
+        return 0, True
+    _check(code, "paged_softmax_attention (tcgen05)")
+    add_launches(int(raw is not None))
+    return _TC_ATTENTION_MIN_TOKENS, min(counts) < _TC_ATTENTION_MIN_TOKENS
 
 
 def head_prepare(proj: torch.Tensor, positions: torch.Tensor | None, *, heads: int, kv_heads: int, dim: int, value_dim: int = 0,

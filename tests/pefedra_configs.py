@@ -61,4 +61,13 @@ WIDE = config([
     layer(turned(2, 2, 112, 16, 0.1, 500), 96),
 ], vocab=128, width=128, eps=1e-5, scale=4.0)
 
+# the sizes that long portions of prompts take to the tcgen05 kernel, with windows shorter and longer than its tiles
+TALL = config([
+    layer(turned(4, 2, 64, 64, 0.12, 90, dims=48), 80),
+    layer(differential(2, 1, 64, 128, 0.15, 140, diff=0.4, factor=2.0), 96),
+    layer(differential(3, 3, 64, 64, 0.12, 33, diff=0.6, dims=24)),
+    layer(turned(2, 1, 128, 128, 0.1, 600), 64),
+    layer(turned(2, 1, 64, 128, 0.12, 65), 112),
+], vocab=80, width=80, eps=1e-5, scale=3.0)
+
 ALL = {"odd": ODD, "ones": ONES, "wide": WIDE}

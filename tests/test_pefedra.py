@@ -245,12 +245,12 @@ def test_long_decoding_over_pages_and_windows(where, engine):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_long_portions(dtype, engine):
+@pytest.mark.parametrize("cfg", [configs.WIDE, configs.TALL], ids=["wide", "tall"])
+def test_long_portions(dtype, cfg, engine):
     """Prompts of some hundred tokens, whole and in two long portions beside a decoding request; then single tokens over a context
     long enough to be shared out over several CTAs."""
     where = f"cuda-{dtype}"
     engine(where)
-    cfg = configs.WIDE
     model, tensors, dtype = make_model(cfg, 23, where, change=_loud)
     reqs = tokens_for(cfg["vocab"], [330, 40], 6)
     exp = expected_of(cfg, tensors, reqs)

@@ -19,7 +19,8 @@ pytestmark = pytest.mark.gpu
 
 # heads, kv heads, key lanes (of a map), value lanes, page size
 SHAPES = [(8, 2, 16, 48, 16), (3, 1, 10, 6, 8), (6, 2, 48, 96, 16), (4, 4, 128, 128, 4), (1, 1, 2, 2, 1), (5, 5, 7, 4, 3), (4, 2, 64, 32, 16),
-          (12, 4, 16, 256, 8), (16, 1, 32, 64, 16), (2, 2, 64, 128, 16), (2, 1, 112, 144, 8), (2, 1, 288, 16, 8)]
+          (12, 4, 16, 256, 8), (16, 1, 32, 64, 16), (2, 2, 64, 128, 16), (2, 1, 112, 144, 8), (2, 1, 288, 16, 8),
+          (6, 2, 64, 64, 32), (4, 1, 64, 128, 8), (4, 2, 128, 128, 16)]
 
 
 def few_rows(ctx, rows, longest):
@@ -46,22 +47,27 @@ def variants(ops, H, V, N, gate):
     ]
 
 
-@pytest.mark.parametrize("general", [False, True])
-@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 2e-2)])
+def use_kernels(monkeypatch, ops, way: str) -> None:
+    """``tcgen05``: as the engine chooses (requests of 128 tokens and more of some sizes on tcgen05); ``mma``: the row kernel also
+    there; ``general``: the kernel for any sizes also where a tensor-core kernel would run."""
+    monkeypatch.setattr(ops, "_FORCE_GENERIC_ATTENTION", way == "general")
+    monkeypatch.setattr(ops, "_TC_ATTENTION_ENABLED", way == "tcgen05")
+
+
+@pytest.mark.parametrize("dtype,tol,way", [(torch.float32, 2e-5, "general"), (torch.bfloat16, 2e-2, "general"), (torch.bfloat16, 2e-2, "mma"),
+                                           (torch.bfloat16, 2e-2, "tcgen05")])
 @pytest.mark.parametrize("H,KV,D,V,page_size", SHAPES)
-def test_maps_turns_and_gates_against_plain(H, KV, D, V, page_size, dtype, tol, general, monkeypatch):
-    """``general``: the kernel for any sizes also where the tensor-core kernel would run (bfloat16, lanes in sixteens).  The
-    result goes into rows with a pitch."""
+def test_maps_turns_and_gates_against_plain(H, KV, D, V, page_size, dtype, tol, way, monkeypatch):
+    """Long and short requests in one step.  The result goes into rows with a pitch."""
     ops = _ops()
-    if general and dtype == torch.float32:
-        pytest.skip("float32 always runs the general kernel")
-    monkeypatch.setattr(ops, "_FORCE_GENERIC_ATTENTION", general)
+    use_kernels(monkeypatch, ops, way)
     torch.manual_seed(H * 100 + D + 2)
-    ctx, table, slots, pages = paged_batch([37, 1, 200, 1300], [5, 1, 200, 2], page_size)
+    ctx, table, slots, pages = paged_batch([37, 1, 340, 1300, 550], [5, 1, 200, 2, 131], page_size)
     N = ctx.num_tokens
     gate = torch.randn(N, H + 4, device=DEV)[:, 2 : 2 + H]
     rows = [4, 5, 205, 207]
     few = few_rows(ctx, rows, 1300)
+    few.context_lens = ctx.context_lens[:4].contiguous()
     for what, more in variants(ops, H, V, N, gate):
         maps = 2 if "differential" in more else 1
         if maps * D > 640:
@@ -80,18 +86,17 @@ def test_maps_turns_and_gates_against_plain(H, KV, D, V, page_size, dtype, tol, 
         close(ops.paged_softmax_attention(q[rows].contiguous(), pool, table, few, **common, **part), full[rows], tol * (3 if maps == 2 else 1), what + ", single tokens")
 
 
-@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("general", [False, True])
-@pytest.mark.parametrize("news", [[600, 1, 1], [1, 1, 1], [64, 2, 1]])
-def test_one_key_at_the_window_decides_in_each_map(news, dtype, general, monkeypatch):
+@pytest.mark.parametrize("dtype,way,D", [(torch.float32, "general", 32), (torch.bfloat16, "general", 32), (torch.bfloat16, "mma", 32), (torch.bfloat16, "tcgen05", 64)])
+@pytest.mark.parametrize("news", [[600, 1, 1], [1, 1, 1], [64, 2, 1], [300, 131, 3]])
+def test_one_key_at_the_window_decides_in_each_map(news, dtype, way, D, monkeypatch):
     """Keys are built from the three base-9 digits of their position (a third of a unit vector per digit), so that a query 66 times
     key j scores 66 on key j and at most 44 on any other visible key.  The first map asks for one key and the second for another:
     with a difference weight of 1/2 and no norm to speak of (eps far above the rows' size, the scale its root) the result is the
     first key's value row less half the second's.  Asked for: the key just inside and just outside a window of 70, keys at page
     borders and the query's own, in either map."""
     ops = _ops()
-    monkeypatch.setattr(ops, "_FORCE_GENERIC_ATTENTION", general)
-    H, KV, D, V, page_size, W = 4, 2, 32, 16, 8, 70
+    use_kernels(monkeypatch, ops, way)
+    H, KV, V, page_size, W = 4, 2, (64 if D == 64 else 16), 8, 70
     lens = [600, 523, 300]
     ctx, table, slots, pages = paged_batch(lens, news, page_size, seed=3)
     pool = torch.zeros(pages, 2, KV, page_size, 2 * D, device=DEV, dtype=dtype)
