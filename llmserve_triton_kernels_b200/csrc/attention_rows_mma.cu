@@ -413,9 +413,9 @@ attention_rows_merge_kernel(const RowsArgs<bf16> a, const float* __restrict__ pa
         const float inv = 1.f / warp_sum(ws * ls);
         const float* po = part_o + first * dv;
         float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};  // eight independent sums a lane: a split's loads are in flight together
-        for (int s = 0; s < splits; ++s) {
+#pragma unroll 4
+        for (int s = 0; s < splits; ++s) {  // (a split without keys for this row has left zeros: nothing is skipped, so that loads run ahead)
             const float w = __shfl_sync(0xffffffffu, ws, s);
-            if (w == 0.f) continue;  // uniform across the warp
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 const int d = lane + 32 * i;
@@ -534,8 +534,8 @@ int launch(const RowsArgs<bf16>& a, int requests, int max_query_len, int splits,
 }  // namespace
 
 // As llm_attention_rows, for bfloat16 with every run of lanes a multiple of 16 and 16-byte aligned rows; dv <= 256.
-// `max_query_len`: the most tokens a request brings (it sizes the grid); skip_from > 0: requests of that many tokens and more are left out.  `splits` > 1 cuts every row tile's keys over
-// that many CTAs; part_o [n_tokens * H * maps * splits * dv] and part_ml [n_tokens * H * maps * splits * 2] (float32) then hold the
+// `max_query_len`: the most tokens a request brings (it sizes the grid); skip_from > 0: requests of that many tokens and more are
+// left out.  `splits` > 1 cuts every row tile's keys over that many CTAs; part_o [n_tokens * H * maps * splits * dv] and part_ml [n_tokens * H * maps * splits * 2] (float32) then hold the
 // partial results until the merge that follows.  Returns LLM_ERR_UNSUPPORTED for shapes it does not take.
 LLM_EXPORT int llm_attention_rows_mma(const void* q0, long long q0_token, long long q0_head, int d0, const void* q1,
                                       long long q1_token, long long q1_head, int d1, void* out, long long out_token,
