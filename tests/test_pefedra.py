@@ -473,6 +473,7 @@ def test_preempted_requests_start_over(where, engine, monkeypatch):
     tensors = random_tensors(llm.model.tensor_specs(), 6, 0.02, torch.bfloat16)
     prompts = list(tokens_for(cfg["vocab"], [9, 11, 7], 18).values())
     outs = llm.generate(prompts, SamplingParams(temperature=0.0, max_new_tokens=16))
+    assert llm.scheduler.stats.preemptions > 0
     for prompt, o in zip(prompts, outs):
         assert len(o.token_ids) == 16
         logits = plain_pefedra.forward(cfg, tensors, prompt + o.token_ids)
