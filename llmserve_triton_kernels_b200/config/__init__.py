@@ -4,6 +4,7 @@ from .kafepel import KafepelConfig  # noqa: F401
 from .nudodra import NudodraConfig  # noqa: F401
 from .pefedra import PefedraConfig  # noqa: F401
 from .tenotar import TenotarConfig  # noqa: F401
+from .zifuzen import ZifuzenConfig  # noqa: F401
 from .registry import (  # noqa: F401
     Architecture,
     architecture_of,

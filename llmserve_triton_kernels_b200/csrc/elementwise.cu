@@ -40,6 +40,53 @@ LLM_EXPORT int llm_embed(const int* ids, const void* table, int table_dtype, flo
     return LLM_ERR_BAD_ARGUMENT;
 }
 
+// embedding with learned positions: out[t, :] = scale * table[ids[t], :] + pos[positions[t], :], 32-bit, and the same row in the
+// compute type in `copy` (or null) for whoever reads the stream itself
+template <typename T, typename TC>
+__global__ void embed_positions_kernel(const int* __restrict__ ids, const T* __restrict__ table, float scale, const int* __restrict__ positions,
+                                       const T* __restrict__ pos, float* __restrict__ out, TC* __restrict__ copy, int hidden, int vocab, int places) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = ids[t], p = positions[t];
+    if (id < 0 || id >= vocab) id = 0;  // launch-side checks reject such ids and positions; never read out of range
+    if (p < 0 || p >= places) p = 0;
+    const T *src = table + (size_t)id * hidden, *at = pos + (size_t)p * hidden;
+    if ((hidden & 3) == 0) {
+        for (int i = threadIdx.x * 4; i < hidden; i += blockDim.x * 4) {
+            float v[4], w[4];
+            load4(src + i, v);
+            load4(at + i, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = fmaf(v[e], scale, w[e]);
+            store4(out + (size_t)t * hidden + i, v);
+            if (copy) store4(copy + (size_t)t * hidden + i, v);
+        }
+    } else {
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+            const float v = fmaf(to_float(src[i]), scale, to_float(at[i]));
+            out[(size_t)t * hidden + i] = v;
+            if (copy) copy[(size_t)t * hidden + i] = from_float<TC>(v);
+        }
+    }
+}
+
+// copy (or null): bfloat16 [n, hidden]
+LLM_EXPORT int llm_embed_positions(const int* ids, const void* table, int table_dtype, float scale, const int* positions, const void* pos,
+                                   float* out, void* copy, int n, int hidden, int vocab, int places, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (vocab <= 0 || places <= 0) return LLM_ERR_BAD_ARGUMENT;
+    const int threads = hidden >= 1024 ? 256 : 128;
+    using bf = __nv_bfloat16;
+    if (table_dtype == LLM_F32)
+        return launch_pdl(embed_positions_kernel<float, bf>, dim3(n), dim3(threads), 0, stream, ids, (const float*)table, scale, positions,
+                          (const float*)pos, out, (bf*)copy, hidden, vocab, places);
+    if (table_dtype == LLM_BF16)
+        return launch_pdl(embed_positions_kernel<bf, bf>, dim3(n), dim3(threads), 0, stream, ids, (const bf*)table, scale, positions, (const bf*)pos,
+                          out, (bf*)copy, hidden, vocab, places);
+    return LLM_ERR_BAD_ARGUMENT;
+}
+
 // ---------------------------------------------------------------------------------------------
 // RMS norm with the residual sum: v = resid[row] (+ delta[row]); resid[row] = v (when all rows are
 // produced); out[i] = v * rsqrt(mean(v^2) + eps) * weight.  `rows` selects input rows (then the
@@ -299,8 +346,14 @@ LLM_EXPORT int llm_rope_kv_write(void* qkv, int dtype, int row_stride, const int
 // ---------------------------------------------------------------------------------------------
 // gated activation: out[t, j] = silu(gate_up[t, j]) * gate_up[t, I + j], in 32-bit
 // ---------------------------------------------------------------------------------------------
+// kind 0: silu, 1: gelu in its tanh form
+__device__ __forceinline__ float gate_act(float v, int kind) {
+    if (kind == 0) return v / (1.f + expf(-v));
+    return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+}
+
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total, const T* __restrict__ bias) {
+__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, size_t total, const T* __restrict__ bias, int kind) {
     pdl_trigger();
     pdl_wait();
     const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -319,7 +372,7 @@ __global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out
                 for (int e = 0; e < 4; ++e) { g[e] += bg[e]; u[e] += bu[e]; }
             }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) g[e] = g[e] / (1.f + expf(-g[e])) * u[e];
+            for (int e = 0; e < 4; ++e) g[e] = gate_act(g[e], kind) * u[e];
             store4(out + i, g);
         }
         return;
@@ -329,22 +382,23 @@ __global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out
         const int j = (int)(i - t * inter);
         const float g = to_float(gate_up[t * 2 * inter + j]) + (bias ? to_float(bias[j]) : 0.f);
         const float u = to_float(gate_up[t * 2 * inter + inter + j]) + (bias ? to_float(bias[inter + j]) : 0.f);
-        out[i] = from_float<T>(g / (1.f + expf(-g)) * u);
+        out[i] = from_float<T>(gate_act(g, kind) * u);
     }
 }
 
-LLM_EXPORT int llm_swiglu(const void* gate_up, void* out, int dtype, int n, int inter, const void* bias, cudaStream_t stream) {
+LLM_EXPORT int llm_swiglu(const void* gate_up, void* out, int dtype, int n, int inter, const void* bias, int kind, cudaStream_t stream) {
     if (n <= 0) return 0;
+    if (kind < 0 || kind > 1) return LLM_ERR_BAD_ARGUMENT;
     const size_t total = (size_t)n * inter;
     const int threads = 256;
     const size_t want = (total / 4 + threads - 1) / threads + 1;
     const size_t most = 148 * 16;  // sixteen blocks an SM of a B200; the kernel's loop strides over what is left
     const int blocks = (int)(want < most ? want : most);
     if (dtype == LLM_F32)
-        return launch_pdl(swiglu_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float*)gate_up, (float*)out, inter, total, (const float*)bias);
+        return launch_pdl(swiglu_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float*)gate_up, (float*)out, inter, total, (const float*)bias, kind);
     if (dtype == LLM_BF16)
         return launch_pdl(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16*)gate_up,
-                          (__nv_bfloat16*)out, inter, total, (const __nv_bfloat16*)bias);
+                          (__nv_bfloat16*)out, inter, total, (const __nv_bfloat16*)bias, kind);
     return LLM_ERR_BAD_ARGUMENT;
 }
 

@@ -16,25 +16,55 @@ namespace {
 // w: [N, E + shared_gate] float32
 // One warp: from a token's logits zr[0 : E (+ 1)] to its row of weights wr; s, c: E floats of scratch each.
 // bias (or null): added to the logits of the E experts first.  shared_gate 2: w[t, E] = 1 (a shared expert without a gate; z has no column E).
+// sigmoid: the scores are s = sigmoid(z) (their sum, with renorm, plus 1e-20).  groups > 0: the experts form so many equal runs of
+// neighbours; a run's score is the sum of its two largest choice scores s + correction, and only experts of the `keep` runs with
+// the largest may be chosen (lowest index among equals); gs: `groups` floats of scratch.
 __device__ __forceinline__ void route_row(const float* zr, const float* __restrict__ correction, float* wr, float* s, float* c, int E, int top,
-                                          float scale, int renorm, int shared_gate, int lane, const float* __restrict__ bias = nullptr) {
+                                          float scale, int renorm, int shared_gate, int lane, const float* __restrict__ bias = nullptr,
+                                          int sigmoid = 0, int groups = 0, int keep = 0, float* gs = nullptr) {
     float m = -FLT_MAX;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e] + (bias ? bias[e] : 0.f));
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) {
-        const float x = expf(zr[e] + (bias ? bias[e] : 0.f) - m);
-        s[e] = x;
-        sum += x;
+    float inv = 1.f;
+    if (sigmoid) {
+        for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-(zr[e] + (bias ? bias[e] : 0.f))));
+    } else {
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e] + (bias ? bias[e] : 0.f));
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) {
+            const float x = expf(zr[e] + (bias ? bias[e] : 0.f) - m);
+            s[e] = x;
+            sum += x;
+        }
+        inv = 1.f / warp_sum(sum);
     }
-    sum = warp_sum(sum);
-    const float inv = 1.f / sum;
     for (int e = lane; e < E; e += 32) {
         s[e] *= inv;
         c[e] = s[e] + (correction ? correction[e] : 0.f);
         wr[e] = 0.f;
     }
     __syncwarp();
+    if (groups > 0) {
+        const int size = E / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float first = -FLT_MAX, second = -FLT_MAX;
+            for (int i = 0; i < size; ++i) {
+                const float v = c[g * size + i];
+                if (v > first) { second = first; first = v; }
+                else if (v > second) second = v;
+            }
+            gs[g] = size > 1 ? first + second : first;
+        }
+        __syncwarp();
+        // a run stays if fewer than `keep` others stand in front of it
+        for (int e = lane; e < E; e += 32) {
+            const int g = e / size;
+            const float mine = gs[g];
+            int ahead = 0;
+            for (int o = 0; o < groups; ++o) ahead += gs[o] > mine || (gs[o] == mine && o < g);
+            if (ahead >= keep) c[e] = -FLT_MAX;
+        }
+        __syncwarp();
+    }
     float chosen_sum = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -FLT_MAX;
@@ -56,7 +86,7 @@ __device__ __forceinline__ void route_row(const float* zr, const float* __restri
         }
         __syncwarp();
     }
-    const float f = renorm ? scale / chosen_sum : scale;
+    const float f = renorm ? scale / (chosen_sum + (sigmoid ? 1e-20f : 0.f)) : scale;
     for (int e = lane; e < E; e += 32)
         if (wr[e] < 0.f) wr[e] = s[e] * f;
     if (shared_gate && lane == 0) wr[E] = shared_gate == 2 ? 1.f : 1.f / (1.f + expf(-zr[E]));
@@ -82,9 +112,9 @@ route_topk_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
 template <typename TX, int TT>
 __global__ void __launch_bounds__(512)
 router_kernel(const TX* __restrict__ x, int ldx, const float* __restrict__ wr, const float* __restrict__ correction, float* __restrict__ out,
-              int N, int K, int E, int top, float scale, int renorm, int shared_gate, const float* __restrict__ bias) {
+              int N, int K, int E, int top, float scale, int renorm, int shared_gate, const float* __restrict__ bias, int sigmoid, int groups, int keep) {
     constexpr int RPW = 4;  // rows of the router matrix a warp sums up at once: what it reads of the tokens serves all four
-    extern __shared__ float sm[];  // z[TT][rows], then per token s[E], c[E]
+    extern __shared__ float sm[];  // z[TT][rows], then per token s[E], c[E], and the scores of runs of experts
     pdl_trigger();
     const int rows = E + (shared_gate == 1), out_w = E + (shared_gate != 0), t0 = blockIdx.x * TT;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
@@ -147,8 +177,9 @@ router_kernel(const TX* __restrict__ x, int ldx, const float* __restrict__ wr, c
     }
     __syncthreads();
     if (warp < TT && t0 + warp < N) {
-        float* s = sm + (size_t)TT * rows + (size_t)warp * 2 * E;
-        route_row(z + warp * rows, correction, out + (size_t)(t0 + warp) * out_w, s, s + E, E, top, scale, renorm, shared_gate, lane, bias);
+        float* s = sm + (size_t)TT * rows + (size_t)warp * (2 * E + groups);
+        route_row(z + warp * rows, correction, out + (size_t)(t0 + warp) * out_w, s, s + E, E, top, scale, renorm, shared_gate, lane, bias, sigmoid, groups,
+                  keep, s + 2 * E);
     }
 }
 
@@ -380,21 +411,22 @@ LLM_EXPORT int llm_route_topk(const float* z, int ldz, const float* correction, 
 }
 
 LLM_EXPORT int llm_router(const void* x, int x_dtype, int ldx, const float* wr, const float* correction, float* out, int N, int K, int E,
-                          int top, float scale, int renorm, int shared_gate, const float* bias, cudaStream_t stream) {
+                          int top, float scale, int renorm, int shared_gate, const float* bias, int sigmoid, int groups, int keep, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (E <= 0 || top < 1 || top > E || E > 2048 || K <= 0 || shared_gate < 0 || shared_gate > 2) return LLM_ERR_BAD_ARGUMENT;
+    if (E <= 0 || top < 1 || top > E || E > 2048 || K <= 0 || shared_gate < 0 || shared_gate > 2 ||
+        groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups || top > keep * (E / groups)))) return LLM_ERR_BAD_ARGUMENT;
     // tokens a CTA: one for steps of few tokens (more CTAs, more loads in flight a warp), two otherwise (three CTAs an SM)
     const int TT = N <= 32 ? 1 : 2;
     const int rows_all = E + (shared_gate == 1 ? 1 : 0);  // rows of the router's matrix (2: the last column of out is the constant 1)
-    const size_t smem = ((size_t)TT * rows_all + (size_t)TT * 2 * E) * sizeof(float);
-    const int groups = (rows_all + 3) / 4;  // of four rows: a warp each, as far as 16 warps go
-    const dim3 grid((N + TT - 1) / TT), block(32 * (groups < 4 ? 4 : groups > 16 ? 16 : groups));
+    const size_t smem = ((size_t)TT * rows_all + (size_t)TT * (2 * E + groups)) * sizeof(float);
+    const int quads = (rows_all + 3) / 4;  // of rows: a warp each, as far as 16 warps go
+    const dim3 grid((N + TT - 1) / TT), block(32 * (quads < 4 ? 4 : quads > 16 ? 16 : quads));
     auto go = [&](auto kernel, auto* xp) -> int {
         if (smem > 48 * 1024) {
             const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (e != cudaSuccess) return (int)e;
         }
-        return launch_pdl(kernel, grid, block, smem, stream, xp, ldx, wr, correction, out, N, K, E, top, scale, renorm, shared_gate, bias);
+        return launch_pdl(kernel, grid, block, smem, stream, xp, ldx, wr, correction, out, N, K, E, top, scale, renorm, shared_gate, bias, sigmoid, groups, keep);
     };
     using bf = __nv_bfloat16;
     if (x_dtype == LLM_F32) return TT == 1 ? go(router_kernel<float, 1>, (const float*)x) : go(router_kernel<float, 2>, (const float*)x);

@@ -12,12 +12,15 @@ namespace {
 
 constexpr int MAX_TAPS = 16;
 
+// what stands behind the sum: 0 nothing, 1 silu
+__device__ __forceinline__ float behind(float v, int act) { return act == 1 ? v / (1.f + expf(-v)) : v; }
+
 // grid (channel blocks, token tiles); a thread a channel, TOKENS rows a CTA
 template <typename TI, int TOKENS>
 __global__ void __launch_bounds__(128)
 short_conv_kernel(const TI* __restrict__ u, int ldu, const float* __restrict__ w, const float* __restrict__ state,
                   const int* __restrict__ state_slots, const int* __restrict__ token_request, const int* __restrict__ cu_tokens,
-                  float* __restrict__ y, int ldy, int N, int C, int taps) {
+                  float* __restrict__ y, int ldy, int N, int C, int taps, int act) {
     pdl_trigger();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     float wt[MAX_TAPS];
@@ -38,7 +41,7 @@ short_conv_kernel(const TI* __restrict__ u, int ldu, const float* __restrict__ w
             const float v = src >= begin ? to_float(u[(size_t)src * ldu + c]) : old[(size_t)(src - begin + back) * C + c];
             acc = fmaf(wt[j], v, acc);
         }
-        y[(size_t)t * ldy + c] = acc;
+        y[(size_t)t * ldy + c] = behind(acc, act);
     }
 }
 
@@ -49,7 +52,7 @@ template <typename TI>
 __global__ void __launch_bounds__(128)
 short_conv4_kernel(const TI* __restrict__ u, int ldu, const float* __restrict__ w, const float* __restrict__ state,
                    const int* __restrict__ state_slots, const int* __restrict__ token_request, const int* __restrict__ cu_tokens,
-                   float* __restrict__ y, int ldy, int N, int C, int taps, int span) {
+                   float* __restrict__ y, int ldy, int N, int C, int taps, int span, int act) {
     constexpr int W = 4;
     pdl_trigger();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -93,6 +96,8 @@ short_conv4_kernel(const TI* __restrict__ u, int ldu, const float* __restrict__ 
         for (int k = 0; k < W; ++k)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[e] = fmaf(wt[k][e], hist[k][e], acc[e]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] = behind(acc[e], act);
         store4(y + (size_t)t * ldy + c, acc);
 #pragma unroll
         for (int k = 0; k < W - 1; ++k)
@@ -131,7 +136,7 @@ short_conv_state_kernel(const TI* __restrict__ u, int ldu, float* __restrict__ s
 template <typename TI>
 __global__ void __launch_bounds__(128)
 short_conv_walk_kernel(const TI* __restrict__ u, int ldu, const float* __restrict__ w, float* __restrict__ state,
-                       const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, float* __restrict__ y, int ldy, int C, int taps) {
+                       const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, float* __restrict__ y, int ldy, int C, int taps, int act) {
     pdl_trigger();
     const int c = blockIdx.x * blockDim.x + threadIdx.x, r = blockIdx.y, back = taps - 1;
     // taps and rows stand at the END of two arrays of MAX_TAPS (tap j at MAX_TAPS - taps + j, zeros in front), so that every
@@ -154,7 +159,7 @@ short_conv_walk_kernel(const TI* __restrict__ u, int ldu, const float* __restric
         float acc = 0.f;
 #pragma unroll
         for (int k = 0; k < MAX_TAPS; ++k) acc = fmaf(wt[k], hist[k], acc);  // the oldest row first, as in the other kernel
-        y[(size_t)t * ldy + c] = acc;
+        y[(size_t)t * ldy + c] = behind(acc, act);
     }
 #pragma unroll
     for (int k = 0; k < MAX_TAPS; ++k)
@@ -164,20 +169,20 @@ short_conv_walk_kernel(const TI* __restrict__ u, int ldu, const float* __restric
 }  // namespace
 
 // u [N, >= C] (float32 or bfloat16, row pitch ldu), w [C, taps] float32, state [slots, taps - 1, C] float32,
-// y [N, C] float32 (row pitch ldy).  taps from 1 to 16 (1: a weight a channel, no state).
+// y [N, C] float32 (row pitch ldy).  taps from 1 to 16 (1: a weight a channel, no state).  act: 0 the sums, 1 their silu.
 LLM_EXPORT int llm_short_conv(const void* u, int dtype, int ldu, const float* w, float* state, const int* state_slots,
                               const int* token_request, const int* cu_tokens, float* y, int ldy, int N, int requests, int C,
-                              int taps, int max_query_len, cudaStream_t stream) {
+                              int taps, int max_query_len, int act, cudaStream_t stream) {
     if (N <= 0 || requests <= 0) return 0;
-    if (C <= 0 || taps < 1 || taps > MAX_TAPS || ldu < C || ldy < C || (taps > 1 && !state) || requests > 65535) return LLM_ERR_BAD_ARGUMENT;
+    if (C <= 0 || taps < 1 || taps > MAX_TAPS || ldu < C || ldy < C || (taps > 1 && !state) || requests > 65535 || act < 0 || act > 1) return LLM_ERR_BAD_ARGUMENT;
     constexpr int TOKENS = 8;
     if (max_query_len > 0 && max_query_len <= 16) {  // few tokens a request: the walk, whose sums have the same order
         const dim3 wgrid((C + 127) / 128, requests);
         if (dtype == LLM_F32)
-            return launch_pdl(short_conv_walk_kernel<float>, wgrid, dim3(128), 0, stream, (const float*)u, ldu, w, state, state_slots, cu_tokens, y, ldy, C, taps);
+            return launch_pdl(short_conv_walk_kernel<float>, wgrid, dim3(128), 0, stream, (const float*)u, ldu, w, state, state_slots, cu_tokens, y, ldy, C, taps, act);
         if (dtype == LLM_BF16)
             return launch_pdl(short_conv_walk_kernel<__nv_bfloat16>, wgrid, dim3(128), 0, stream, (const __nv_bfloat16*)u, ldu, w, state, state_slots,
-                              cu_tokens, y, ldy, C, taps);
+                              cu_tokens, y, ldy, C, taps, act);
         return LLM_ERR_BAD_ARGUMENT;
     }
     const dim3 block(128), grid((C + 127) / 128, (N + TOKENS - 1) / TOKENS);
@@ -191,20 +196,20 @@ LLM_EXPORT int llm_short_conv(const void* u, int dtype, int ldu, const float* w,
         if (g4.y > 65535) return LLM_ERR_UNSUPPORTED;
         if (dtype == LLM_F32)
             code = launch_pdl(short_conv4_kernel<float>, g4, block, 0, stream, (const float*)u, ldu, w, (const float*)state, state_slots, token_request,
-                              cu_tokens, y, ldy, N, C, taps, span);
+                              cu_tokens, y, ldy, N, C, taps, span, act);
         else if (dtype == LLM_BF16)
             code = launch_pdl(short_conv4_kernel<__nv_bfloat16>, g4, block, 0, stream, (const __nv_bfloat16*)u, ldu, w, (const float*)state, state_slots,
-                              token_request, cu_tokens, y, ldy, N, C, taps, span);
+                              token_request, cu_tokens, y, ldy, N, C, taps, span, act);
         else
             return LLM_ERR_BAD_ARGUMENT;
     } else if (grid.y > 65535)
         return LLM_ERR_UNSUPPORTED;
     else if (dtype == LLM_F32)
         code = launch_pdl(short_conv_kernel<float, TOKENS>, grid, block, 0, stream, (const float*)u, ldu, w, (const float*)state, state_slots,
-                          token_request, cu_tokens, y, ldy, N, C, taps);
+                          token_request, cu_tokens, y, ldy, N, C, taps, act);
     else if (dtype == LLM_BF16)
         code = launch_pdl(short_conv_kernel<__nv_bfloat16, TOKENS>, grid, block, 0, stream, (const __nv_bfloat16*)u, ldu, w,
-                          (const float*)state, state_slots, token_request, cu_tokens, y, ldy, N, C, taps);
+                          (const float*)state, state_slots, token_request, cu_tokens, y, ldy, N, C, taps, act);
     else
         return LLM_ERR_BAD_ARGUMENT;
     if (code != 0 || taps == 1) return code;

@@ -174,7 +174,8 @@ __global__ void stream_inject_kernel(float* __restrict__ resid, const TD* __rest
 }
 
 // ---------------------------------------------------------------------------------------------
-// one-input functions of a matrix with a row pitch: 0 relu(v)^2, 1 gelu (tanh form), 2 alpha * v, 3 silu, 4 gelu (erf form)
+// one-input functions of a matrix with a row pitch: 0 relu(v)^2, 1 gelu (tanh form), 2 alpha * v, 3 silu, 4 gelu (erf form),
+// 5 alpha * tanh(v / alpha)
 // ---------------------------------------------------------------------------------------------
 __device__ __forceinline__ float unary_of(float v, int kind, float alpha) {
     switch (kind) {
@@ -182,6 +183,7 @@ __device__ __forceinline__ float unary_of(float v, int kind, float alpha) {
         case 1: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
         case 2: return alpha * v;
         case 4: return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+        case 5: return alpha * tanhf(v / alpha);
         default: return v * sigmoid_f(v);
     }
 }
@@ -250,7 +252,8 @@ int unary_wide(const T* x, int ldx, T* out, int ldo, int rows, int cols, int kin
         case 1: return go(unary_wide_kernel<T, 1>);
         case 2: return go(unary_wide_kernel<T, 2>);
         case 3: return go(unary_wide_kernel<T, 3>);
-        default: return go(unary_wide_kernel<T, 4>);
+        case 4: return go(unary_wide_kernel<T, 4>);
+        default: return go(unary_wide_kernel<T, 5>);
     }
 }
 
@@ -344,7 +347,7 @@ LLM_EXPORT int llm_stream_inject(float* resid, const void* delta, int delta_dtyp
 LLM_EXPORT int llm_unary(const void* x, int ldx, void* out, int ldo, int dtype, int rows, int cols, int kind, float alpha,
                          cudaStream_t stream) {
     if (rows <= 0 || cols <= 0) return 0;
-    if (ldx < cols || ldo < cols || kind < 0 || kind > 4) return LLM_ERR_BAD_ARGUMENT;
+    if (ldx < cols || ldo < cols || kind < 0 || kind > 5) return LLM_ERR_BAD_ARGUMENT;
     const size_t total = (size_t)rows * cols;
     if (((cols | ldx | ldo) & 7) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)out & 15) == 0) {
         if (dtype == LLM_F32) return unary_wide<float>((const float*)x, ldx, (float*)out, ldo, rows, cols, kind, alpha, stream);

@@ -44,6 +44,7 @@ class Model:
         self._named_parts.append((plan.final_norm.prefix, self.final_norm))
         self.embedding: torch.Tensor | None = None
         self.head: torch.Tensor | None = None
+        self.position_table: torch.Tensor | None = None
         self._injections = {inj.before: inj for inj in plan.injections}
         self._vectors: dict[str, torch.Tensor] = {}  # the plan's extra tensors, 32-bit
         # a function (entry index, residual stream [N, hidden] with everything added) that is called after every
@@ -55,6 +56,8 @@ class Model:
         """Every tensor of the checkpoint by its full name."""
         plan = self.plan
         specs = {plan.embedding: TensorSpec((plan.vocab_size, plan.hidden_size))}
+        if plan.positions is not None:
+            specs[plan.positions] = TensorSpec((plan.max_positions, plan.hidden_size))
         for prefix, part in self._named_parts:
             for local, spec in part.tensors().items():
                 name = prefix + local
@@ -76,6 +79,8 @@ class Model:
     def bind(self, tensors: dict[str, torch.Tensor]) -> None:
         plan = self.plan
         self.embedding = tensors[plan.embedding].to(device=self.device, dtype=self.dtype).contiguous()
+        if plan.positions is not None:
+            self.position_table = tensors[plan.positions].to(device=self.device, dtype=self.dtype).contiguous()
         if plan.head is None:
             self.head = self.embedding
         else:
@@ -127,8 +132,9 @@ class Model:
         shared = getattr(ctx, "shared", None)
         if shared is not None:
             shared.clear()  # nothing of an earlier pass over this context is handed on
-        resid = self.embed_tokens(ctx)
-        pending = None
+        resid, pending = self.embed_tokens(ctx), None
+        if isinstance(resid, tuple):
+            resid, pending = resid
         order = self.plan.schedule
         for i, run in enumerate(order):
             if i in self._injections:
@@ -190,12 +196,18 @@ class Model:
     def embed_tokens(self, ctx) -> torch.Tensor:
         """The residual stream that the first layer meets: the tokens' rows of the table, in 32-bit ``[N, hidden]``.
         An architecture that scales or otherwise prepares its embeddings overrides this in a subclass that it names
-        when it registers (``register_architecture(..., model_class=...)``)."""
+        when it registers (``register_architecture(..., model_class=...)``).  May return a pair: the stream, and what the
+        first block takes as pending (the same rows in the compute type, ``ops.StreamCopy``)."""
         if self.plan.streams is not None:
             x = ops.embed(ctx.token_ids, self.embedding, copies=self.plan.streams)  # [streams, N, hidden]
             if self.plan.embedding_scale != 1.0:
                 ops.unary(x.view(-1, x.shape[-1]), "scale", self.plan.embedding_scale, inplace=True)
             return x
+        if self.position_table is not None:
+            wants_copy = self.dtype != torch.float32 and 0 not in self._injections and self.blocks[self.plan.schedule[0].layer].reads_stream
+            x, copy = ops.embed_positions(ctx.token_ids, self.embedding, ctx.positions, self.position_table, self.plan.embedding_scale,
+                                          copy_dtype=self.dtype if wants_copy else None)
+            return x if copy is None else (x, ops.StreamCopy(copy))
         x = ops.embed(ctx.token_ids, self.embedding)
         if self.plan.embedding_scale != 1.0:
             ops.unary(x, "scale", self.plan.embedding_scale, inplace=True)
@@ -207,4 +219,6 @@ class Model:
         logits = ops.linear(x, self.head, out_dtype=torch.float32)
         if self.plan.logit_scale != 1.0:
             ops.unary(logits, "scale", self.plan.logit_scale, inplace=True)
+        if self.plan.logit_softcap is not None:
+            ops.unary(logits, "softcap", self.plan.logit_softcap, inplace=True)
         return logits

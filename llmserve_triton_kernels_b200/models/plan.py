@@ -85,6 +85,8 @@ class ModelPlan:
     extra_tensors: tuple[tuple[str, tuple[int, ...]], ...] = ()  # (name, shape) of tensors that belong to no part
     logit_scale: float = 1.0  # the logits are the output matrix's product times this
     embedding_scale: float = 1.0  # the residual stream starts as the tokens' rows of the table times this
+    positions: str | None = None  # tensor name of a table [max_positions, hidden] whose row p is added to the embedding of a token at position p
+    logit_softcap: float | None = None  # the logits z (after logit_scale) become cap * tanh(z / cap)
     streams: int | None = None  # the residual stream is kept in this many copies [streams, N, hidden], all equal at the start (None: one plain stream)
 
     def __post_init__(self) -> None:
@@ -98,6 +100,8 @@ class ModelPlan:
                     raise ValueError(f"schedule entry {i} reads the cache of entry {run.cache_of}, which keeps none itself")
         if self.streams is not None and (self.streams < 1 or self.injections):
             raise ValueError("a stream kept in copies needs at least one copy, and takes nothing up between its layers")
+        if self.positions is not None and (self.max_positions is None or self.streams is not None):
+            raise ValueError("a table of positions has a row for each of max_positions places, and feeds one plain stream")
         declared = {name for name, _ in self.extra_tensors}
         seen = set()
         for inj in self.injections:

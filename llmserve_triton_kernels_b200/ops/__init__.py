@@ -25,7 +25,8 @@ _SIGNATURES = {
     "llm_embed": [_vp, _vp, _i, _vp, _i, _i, _i, _vp],
     "llm_rmsnorm": [_vp, _vp, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
     "llm_rope_kv_write": [_vp, _i, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
-    "llm_swiglu": [_vp, _vp, _i, _i, _i, _vp, _vp],
+    "llm_embed_positions": [_vp, _vp, _i, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "llm_swiglu": [_vp, _vp, _i, _i, _i, _vp, _i, _vp],
     "llm_add_bias": [_vp, _i, _i, _i, _i, _vp, _vp],
     "llm_fetch_words": [_vp, _vp, _vp, _i, _i, _vp],
     "llm_set_error_flag": [_vp],
@@ -72,11 +73,14 @@ _SIGNATURES = {
     "llm_hyper_mix_norm": [_vp, _vp, _vp, _vp, _vp, _f, _f, _f, _f, _i, _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "llm_head_prepare": [_vp, _i, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _f, _i, _vp, _i, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _i, _vp, _vp, _vp],
     "llm_shift_norm": [_vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
-    "llm_short_conv": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "llm_short_conv": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "llm_row_norm": [_vp, _vp, _f, _vp, _vp, _f, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "llm_delta_scan": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
+    "llm_delta_step": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp],
     "llm_row_rmsnorm": [_vp, _i, _i, _vp, _f, _vp, _i, _i, _i, _i, _vp],
     "llm_gated_scan": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _f, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "llm_expert_gated_act": [_vp, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _f, _f, _vp],
-    "llm_router": [_vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _vp, _vp],
+    "llm_router": [_vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _vp, _i, _i, _i, _vp],
     "llm_route_topk": [_vp, _i, _vp, _vp, _i, _i, _i, _f, _i, _i, _vp],
     "llm_expert_act_scale": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "llm_branch_sum_norm": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _vp],
@@ -212,6 +216,25 @@ def embed(ids: torch.Tensor, table: torch.Tensor, copies: int | None = None) -> 
     out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
     _check(_launch("llm_embed", _ptr(ids), _ptr(table), _code(table.dtype), _ptr(out), n, hidden, vocab, _stream()), "embed")
     return out
+
+
+def embed_positions(ids: torch.Tensor, table: torch.Tensor, positions: torch.Tensor, pos: torch.Tensor, scale: float = 1.0,
+                    copy_dtype: torch.dtype | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """``scale * table[ids] + pos[positions]`` in 32-bit, ``[N, hidden]`` (``table [vocab, hidden]`` and the learned vectors
+    ``pos [places, hidden]`` of one type); with ``copy_dtype`` bfloat16 also the same rows rounded to it, for whoever reads the
+    stream itself."""
+    _i32(ids, "ids")
+    _i32(positions, "positions")
+    _need(table.dim() == 2 and table.is_contiguous() and pos.dim() == 2 and pos.is_contiguous() and pos.dtype == table.dtype
+          and pos.shape[1] == table.shape[1] and positions.numel() == ids.numel(), "embed_positions: two contiguous tables of one type and row size")
+    _need(copy_dtype in (None, torch.bfloat16), "embed_positions: the copy is bfloat16")
+    n, (vocab, hidden) = ids.numel(), table.shape
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    copy = torch.empty((n, hidden), dtype=copy_dtype, device=table.device) if copy_dtype is not None else None
+    code = _launch("llm_embed_positions", _ptr(ids), _ptr(table), _code(table.dtype), float(scale), _ptr(positions), _ptr(pos), _ptr(out), _ptr(copy),
+                   n, hidden, vocab, pos.shape[0], _stream())
+    _check(code, "embed_positions")
+    return out, copy
 
 
 def rmsnorm(
@@ -381,6 +404,21 @@ class WeightedSum:
         return out
 
 
+class StreamCopy:
+    """Nothing is pending: the stream holds everything, and ``rows [N, hidden]`` are its rows in the compute type, as the kernel
+    that made them left them for a block whose parts read the stream itself."""
+
+    def __init__(self, rows: torch.Tensor):
+        self.rows = rows
+
+
+class Biased:
+    """A part's result ``tensor [N, hidden]`` whose bias ``[hidden]`` (float32) is still to be added by the kernel that takes it up."""
+
+    def __init__(self, tensor: torch.Tensor, bias: torch.Tensor):
+        self.tensor, self.bias = tensor, bias
+
+
 class StreamUpdate:
     """What a part between hyper-connections returned, not yet taken up by the copies of the stream: ``result`` (a
     float32 tensor ``[N, width]`` or a :class:`WeightedSum`), and the part's ``mix [S, S]`` (from, to) and ``take [S]``:
@@ -403,7 +441,7 @@ def split_pending(pending) -> tuple[torch.Tensor | None, float]:
     """``(what is still to be added to the stream or None, its factor)`` of what a part or a block returned."""
     if isinstance(pending, (BranchSum, WeightedSum)):
         return pending.materialize(), 1.0
-    if pending is None or pending is ADDED:
+    if pending is None or pending is ADDED or isinstance(pending, StreamCopy):
         return None, 1.0
     if isinstance(pending, Scaled):
         return pending.tensor, pending.alpha
@@ -807,14 +845,18 @@ def _split_counters(device, n: int) -> torch.Tensor:
     return buf
 
 
-def swiglu(gate_up: torch.Tensor, bias: torch.Tensor | None = None) -> torch.Tensor:
-    """``silu(gate_up[:, :I]) * gate_up[:, I:]`` computed in 32-bit -> ``[N, I]``.  ``bias`` (``[2 I]``, of the rows' type,
-    laid out like a row): the two projections' biases, added in 32-bit on the way in."""
+_GATED_KINDS = {"silu": 0, "gelu_tanh": 1}
+
+
+def swiglu(gate_up: torch.Tensor, bias: torch.Tensor | None = None, activation: str = "silu") -> torch.Tensor:
+    """``act(gate_up[:, :I]) * gate_up[:, I:]`` computed in 32-bit -> ``[N, I]``, ``act`` silu or gelu in its tanh form.  ``bias``
+    (``[2 I]``, of the rows' type, laid out like a row): the two projections' biases, added in 32-bit on the way in."""
+    _need(activation in _GATED_KINDS, f"swiglu: no activation {activation!r}; known: {sorted(_GATED_KINDS)}")
     _need(gate_up.dim() == 2 and gate_up.is_contiguous() and gate_up.shape[1] % 2 == 0, "gate_up must be a contiguous [N, 2 I] matrix")
     _need(bias is None or (bias.dtype == gate_up.dtype and bias.is_contiguous() and bias.numel() == gate_up.shape[1]), "swiglu: the bias is [2 I] of the rows' type")
     n, inter = gate_up.shape[0], gate_up.shape[1] // 2
     out = torch.empty((n, inter), dtype=gate_up.dtype, device=gate_up.device)
-    _check(_launch("llm_swiglu", _ptr(gate_up), _ptr(out), _code(gate_up.dtype), n, inter, _ptr(bias), _stream()), "swiglu")
+    _check(_launch("llm_swiglu", _ptr(gate_up), _ptr(out), _code(gate_up.dtype), n, inter, _ptr(bias), _GATED_KINDS[activation], _stream()), "swiglu")
     return out
 
 
@@ -886,7 +928,7 @@ def sample(
 # ------------------------------------------------------------------------------------------------
 # Operations of layers that normalise in groups, scale their contributions, gate their outputs, keep a recurrent
 # state, or attend over a latent (csrc/stream_ops.cu, recurrent.cu, cache_write.cu, attention_generic.cu).
-_UNARY_KINDS = {"relu2": 0, "gelu_tanh": 1, "scale": 2, "silu": 3, "gelu": 4}
+_UNARY_KINDS = {"relu2": 0, "gelu_tanh": 1, "scale": 2, "silu": 3, "gelu": 4, "softcap": 5}
 _GATE_KINDS = {"sigmoid": 0, "silu": 1}
 
 
@@ -949,7 +991,7 @@ def stream_inject(
 
 def unary(x: torch.Tensor, kind: str, alpha: float = 1.0, inplace: bool = False, out: torch.Tensor | None = None) -> torch.Tensor:
     """A one-input function of every element, computed in 32-bit: ``relu2`` (the square of relu), ``gelu_tanh``, ``gelu``
-    (the erf form), ``silu``, or ``scale`` (``alpha * x``).  ``x [N, C]`` and ``out`` may have a row pitch."""
+    (the erf form), ``silu``, ``scale`` (``alpha * x``) or ``softcap`` (``alpha * tanh(x / alpha)``).  ``x [N, C]`` and ``out`` may have a row pitch."""
     _need(kind in _UNARY_KINDS, f"no one-input function {kind!r}; known: {sorted(_UNARY_KINDS)}")
     _need(x.dim() == 2 and x.stride(1) == 1, "unary: a matrix with unit inner stride")
     if out is None:
@@ -1730,12 +1772,16 @@ def route_topk(z: torch.Tensor, correction: torch.Tensor | None, experts: int, t
 
 
 def route(x: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor | None, experts: int, top: int, scale: float = 1.0,
-          renormalize: bool = False, shared_gate: bool = False, bias: torch.Tensor | None = None, shared_one: bool = False) -> torch.Tensor:
+          renormalize: bool = False, shared_gate: bool = False, bias: torch.Tensor | None = None, shared_one: bool = False,
+          scores: str = "softmax", groups: tuple[int, int] | None = None) -> torch.Tensor:
     """The router's 32-bit product and :func:`route_topk` in one kernel: ``x [N, K]`` (float32 or bfloat16, read as 32-bit),
     ``w_router [experts (+ 1), K]`` float32 (its last row the shared expert's gate with ``shared_gate``).  A token's sums
     are added in an order of their own, whatever else the step holds.  ``bias`` (float32 ``[experts]``) is added to the
     logits before anything else.  ``shared_one``: a last column of ones (a shared expert without a gate; the router has no
     row for it).  With ``renormalize`` and no correction the weights are the softmax over the chosen logits alone.
+    ``scores="sigmoid"``: ``s = sigmoid(z)`` expert by expert (the chosen ones' sum, with ``renormalize``, plus 1e-20).
+    ``groups = (count, keep)``: the experts form ``count`` equal runs of neighbours; a run's score is the sum of its two largest
+    ``s + correction``, and only experts of the ``keep`` best runs can be chosen (the lowest index among equals).
     Returns ``[N, experts (+ 1)]`` float32."""
     _need(not (shared_gate and shared_one), "route: a shared expert has a gate or the weight one, not both")
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == experts), "route: bias is float32 [experts]")
@@ -1743,9 +1789,13 @@ def route(x: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor | No
     _need(x.dim() == 2 and x.stride(1) == 1 and w_router.dtype == torch.float32 and w_router.is_contiguous()
           and tuple(w_router.shape) == (rows, x.shape[1]), "route: x [N, K], w_router float32 [experts (+ 1), K]")
     _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == experts), "route: correction is float32 [experts]")
+    _need(scores in ("softmax", "sigmoid"), f"route: scores are softmax or sigmoid, not {scores!r}")
+    count, keep = (0, 0) if groups is None else (int(groups[0]), int(groups[1]))
+    _need(groups is None or (1 <= keep <= count and experts % count == 0 and top <= keep * (experts // count)), f"route: {groups} groups of {experts} experts")
     out = torch.empty((x.shape[0], rows + int(shared_one)), dtype=torch.float32, device=x.device)
     code = _launch("llm_router", _ptr(x), _code(x.dtype), x.stride(0), _ptr(w_router), _ptr(correction), _ptr(out), x.shape[0], x.shape[1],
-                   experts, top, float(scale), int(renormalize), 2 if shared_one else int(shared_gate), _ptr(bias), _stream())
+                   experts, top, float(scale), int(renormalize), 2 if shared_one else int(shared_gate), _ptr(bias),
+                   int(scores == "sigmoid"), count, keep, _stream())
     _check(code, "route")
     return out
 
@@ -1803,16 +1853,19 @@ def branch_sum_rmsnorm(pending: BranchSum, resid: torch.Tensor, weight: torch.Te
 # ------------------------------------------------------------------------------------------------
 # Operations of layers whose projections pass a short convolution over time, and of norms on a part of a stacked
 # projection (csrc/short_conv.cu, stream_ops.cu).
-def short_conv(u: torch.Tensor, weight: torch.Tensor, states: torch.Tensor | None, state_slots: torch.Tensor, ctx, channels: int | None = None) -> torch.Tensor:
+def short_conv(u: torch.Tensor, weight: torch.Tensor, states: torch.Tensor | None, state_slots: torch.Tensor, ctx, channels: int | None = None,
+               activation: str | None = None) -> torch.Tensor:
     """A causal convolution over time on each of the first ``channels`` columns of ``u [N, >= channels]`` (rows may have a
     pitch): ``y_t = sum_j weight[:, j] * u_(t - taps + 1 + j)`` within every request, ``weight [channels, taps]`` float32.
     What lies before a request's first row of this step is read from ``states[state_slots[r]]`` (``[slots, taps - 1,
     channels]`` float32: the last rows that earlier steps brought, zeros at a request's start), which is then moved on
     to the last ``taps - 1`` rows after this step.  A step in which no request brings more than 16 tokens
     (``ctx.max_query_len``) is one launch that walks every request's rows; the sums have the same order either way.
+    ``activation``: None or ``silu``, of the sums.
     Returns ``y [N, channels]`` float32."""
     c = int(channels) if channels is not None else weight.shape[0]
     taps = weight.shape[1]
+    _need(activation in (None, "silu"), f"short_conv: no activation {activation!r}")
     _need(u.dim() == 2 and u.stride(1) == 1 and u.shape[1] >= c, "short_conv: u [N, >= channels]")
     _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.shape[0] == c and 1 <= taps <= 16, "short_conv: weight is float32 [channels, taps], taps up to 16")
     if taps > 1:
@@ -1820,7 +1873,7 @@ def short_conv(u: torch.Tensor, weight: torch.Tensor, states: torch.Tensor | Non
     _i32(state_slots, "state_slots")
     out = torch.empty((u.shape[0], c), dtype=torch.float32, device=u.device)
     code = _launch("llm_short_conv", _ptr(u), _code(u.dtype), u.stride(0), _ptr(weight), _ptr(states), _ptr(state_slots), _ptr(ctx.token_request),
-                   _ptr(ctx.cu_tokens), _ptr(out), out.stride(0), u.shape[0], ctx.num_requests, c, taps, int(getattr(ctx, "max_query_len", 0) or 0), _stream())
+                   _ptr(ctx.cu_tokens), _ptr(out), out.stride(0), u.shape[0], ctx.num_requests, c, taps, int(getattr(ctx, "max_query_len", 0) or 0), int(activation == "silu"), _stream())
     _check(code, "short_conv")
     add_launches(int(taps > 1 and not 0 < int(getattr(ctx, "max_query_len", 0) or 0) <= 16))
     return out
@@ -1837,3 +1890,88 @@ def row_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: to
                    x.shape[0], x.shape[1], _stream())
     _check(code, "row_rmsnorm")
     return out
+
+
+# ------------------------------------------------------------------------------------------------
+# Operations of layers that norm what a part returns, and of the gated delta rule (csrc/post_norm.cu, delta_rule.cu).
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, delta: torch.Tensor | None = None, alpha: float = 1.0,
+               rows: torch.Tensor | None = None, out_dtype: torch.dtype = torch.float32, center: bool = True) -> torch.Tensor:
+    """``v = x + alpha * delta``; returns ``(v - mean) / sqrt(mean((v - mean)^2) + eps) * weight`` in ``out_dtype`` (``center=False``: the
+    mean is taken as 0, the RMS form).  Without ``rows`` the sum is written back to ``x``; with ``rows`` (int32) only those rows
+    are produced and ``x`` is left as it was."""
+    _need(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), "layer_norm: the rows are contiguous float32 [N, C]")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == x.shape[1], "layer_norm: the weight is float32 [C]")
+    _need(delta is None or (delta.dtype == torch.float32 and delta.shape == x.shape and delta.is_contiguous()), "layer_norm: delta is float32 of the rows' shape")
+    if rows is not None:
+        _i32(rows, "rows")
+    n_out = x.shape[0] if rows is None else rows.numel()
+    out = torch.empty((n_out, x.shape[1]), dtype=out_dtype, device=x.device)
+    code = _launch("llm_row_norm", _ptr(x), _ptr(delta), float(alpha), None, _ptr(weight), float(eps), int(center), _ptr(rows), None, _ptr(out),
+                   _code(out_dtype), n_out, x.shape[1], _stream())
+    _check(code, "layer_norm")
+    return out
+
+
+def post_norm_add(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, bias: torch.Tensor | None = None,
+                  copy_dtype: torch.dtype | None = None, center: bool = True) -> torch.Tensor | None:
+    """``stream += norm(y + bias) * weight`` row by row, in place, one kernel: a layer norm (``center=False``: an RMS norm) of what a
+    part returned, ``y [N, C]`` float32 (``bias [C]`` float32 or None).  With ``copy_dtype`` the stream's new rows are returned in
+    that type as well."""
+    for t in (stream, y):
+        _need(t.dtype == torch.float32 and t.dim() == 2 and t.is_contiguous() and t.shape == stream.shape, "post_norm_add: contiguous float32 [N, C]")
+    for t in (weight, bias):
+        _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == y.shape[1]), "post_norm_add: weight and bias are float32 [C]")
+    copy = torch.empty(y.shape, dtype=copy_dtype, device=y.device) if copy_dtype is not None else None
+    code = _launch("llm_row_norm", _ptr(y), None, 1.0, _ptr(bias), _ptr(weight), float(eps), int(center), None, _ptr(stream), _ptr(copy),
+                   _code(copy_dtype or torch.float32), y.shape[0], y.shape[1], _stream())
+    _check(code, "post_norm_add")
+    return copy
+
+
+_DELTA_STEP_TOKENS = 16  # up to so many tokens a request the gated delta rule is one launch that holds a head's state in registers
+_DELTA_BLOCK, _DELTA_COEF = 8, 144  # tokens a block of the scan, and the factors it has for each head
+
+
+def delta_rule(y: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, gate: torch.Tensor,
+               weight: torch.Tensor, eps: float, states: torch.Tensor, state_slots: torch.Tensor, ctx, *, heads: int, kv_heads: int,
+               dim: int, value_dim: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """The gated delta rule over every request's new tokens, from and to ``states[state_slots[r]]`` (``[slots, heads, dim,
+    value_dim]`` float32).  ``y [N, 2 * kv_heads * dim + heads * value_dim]`` float32 holds q, k and v; ``beta`` and ``decay [N, >=
+    heads]`` float32 the logits of the step sizes and decays; ``a_log``, ``dt_bias [heads]`` float32.  With q, k made unit vectors
+    (``x / sqrt(sum x^2 + 1e-6)``, q times ``dim^(-1/2)``; head h reads q/k head ``h // (heads / kv_heads)``),
+    ``b = sigmoid(beta)`` and ``g = exp(-exp(a_log) * softplus(decay + dt_bias))`` per head
+
+        S <- g S        u = b (v - S^T k)        S <- S + k u^T        o = S^T q
+
+    and the result is ``o / sqrt(mean(o^2) + eps) * weight * silu(gate)`` over each head's lanes (``weight [value_dim]`` float32,
+    ``gate [N, >= heads * value_dim]`` float32), ``[N, heads * value_dim]`` in ``out_dtype``.  Everything is 32-bit.  ``y`` may be
+    overwritten."""
+    n = y.shape[0]
+    qk, vv = kv_heads * dim, heads * value_dim
+    _need(heads % kv_heads == 0 and y.dtype == torch.float32 and y.dim() == 2 and y.stride(1) == 1 and y.shape[1] >= 2 * qk + vv, "delta_rule: y rows hold q, k and v")
+    for t, w in ((beta, heads), (decay, heads), (gate, vv)):
+        _need(t.dtype == torch.float32 and t.dim() == 2 and t.stride(1) == 1 and t.shape[0] == n and t.shape[1] >= w, "delta_rule: step sizes, decays and the gate are float32 rows")
+    for t, w in ((a_log, heads), (dt_bias, heads), (weight, value_dim)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == w, "delta_rule: A_log and dt_bias are float32 [heads], the norm weight [value_dim]")
+    _need(states.dtype == torch.float32 and states.is_contiguous() and tuple(states.shape[1:]) == (heads, dim, value_dim), "delta_rule: states [slots, heads, dim, value_dim] float32")
+    _i32(state_slots, "state_slots")
+    requests, longest = ctx.num_requests, ctx.max_query_len
+    if longest <= _DELTA_STEP_TOKENS:
+        out = torch.empty((n, vv), dtype=out_dtype, device=y.device)
+        code = _launch("llm_delta_step", _ptr(y), y.stride(0), _ptr(beta), beta.stride(0), _ptr(decay), decay.stride(0), _ptr(a_log), _ptr(dt_bias),
+                       _ptr(gate), gate.stride(0), _ptr(weight), _ptr(states), _ptr(state_slots), _ptr(ctx.cu_tokens), _ptr(out), _code(out_dtype),
+                       out.stride(0), requests, kv_heads, heads, dim, value_dim, dim ** -0.5, float(eps), _stream())
+        if code != 10002:
+            _check(code, "delta_rule (few tokens)")
+            return out
+        add_launches(-1)  # a head's state does not fit one CTA: the way for prompts below
+    coef = torch.empty(((n // _DELTA_BLOCK + requests + 1) * heads * _DELTA_COEF,), dtype=torch.float32, device=y.device)
+    o = torch.empty((n, heads, value_dim), dtype=torch.float32, device=y.device)
+    cols = 64 if dim <= 64 else 32  # columns of the state a CTA takes where there are CTAs enough
+    wide = -(-value_dim // cols) * heads * requests >= 2 * _sm_count()
+    code = _launch("llm_delta_scan", _ptr(y), y.stride(0), _ptr(beta), beta.stride(0), _ptr(decay), decay.stride(0), _ptr(a_log), _ptr(dt_bias), _ptr(states),
+                   _ptr(state_slots), _ptr(ctx.cu_tokens), _ptr(coef), _ptr(o), requests, longest, kv_heads, heads, dim, value_dim, dim ** -0.5,
+                   int(wide), _stream())
+    add_launches(1)
+    _check(code, "delta_rule")
+    return head_norm_gate(o, gate[:, :vv], eps, "silu", out_dtype=out_dtype, weight=weight)

@@ -9,7 +9,7 @@ name, and is handed them once they are loaded.
 Interfaces (what a new part must provide):
 
 * every part: ``tensors() -> {local name: TensorSpec}`` and ``bind(tensors, dtype, device)``;
-* ``Norm``: ``forward(x) -> y`` (and optionally the fused ``add_forward``);
+* ``Norm``: ``forward(x) -> y`` (and optionally the fused ``add_forward``; ``after_forward`` to stand behind a part);
 * ``PositionEncoding``: ``apply(q, k, positions)`` in place on ``[N, heads, head_dim]`` views;
 * ``Mixer``: ``cache_spec()`` saying what it keeps per request (pages of keys and values, a
   slot of fixed-size state, or nothing) and ``forward(x, ctx, cache) -> delta``;
@@ -109,6 +109,9 @@ class Part:
     # ``output_width`` is the inner size of that product, ``release_output_matrix()`` hands the matrix ``[hidden, output_width]``
     # over (once, after ``bind``), and ``forward(..., into=view)`` leaves the product's input rows in ``view [N, output_width]``.
     joins_output = False
+    # True for a feed-forward that, called with ``leave_bias=True``, returns its last product's bias beside the product
+    # (``ops.Biased``), for a kernel that takes the result up anyway
+    leaves_bias = False
 
     def tensors(self) -> dict[str, TensorSpec]:
         return {}
@@ -178,6 +181,9 @@ class Block(Part):
 
     category = "block"
     roles: dict[str, str] = {}
+    # True if the block's first part reads the stream itself: whoever makes the stream may hand its rows in the compute type over
+    # with it (``ops.StreamCopy``)
+    reads_stream = False
     # every contribution of this block's parts enters the residual stream times this
     residual_scale: float = 1.0
 

@@ -204,6 +204,70 @@ class ParallelMixerOnlyBlock(ParallelBlock):
         super().__init__(mixer_norm, mixer, None, None, hidden_size, token_shift, shift_name)
 
 
+class PostNormBlock(Block):
+    """A layer whose parts read the stream itself and whose norms stand behind them:
+
+        x <- x + norm1(mixer(x))        x <- x + norm2(feed_forward(x))
+
+    A part's product leaves its result in 32-bit; one kernel adds a bias that the part left for it (``Part.leaves_bias``), norms,
+    sums into the stream and writes the stream's new rows in the compute type for the part behind (``ops.StreamCopy``).  In 32-bit
+    the parts read the stream's own rows."""
+
+    roles = {"mixer": "mixer", "mixer_norm": "norm", "feed_forward": "feed_forward", "ff_norm": "norm"}
+    reads_stream = True
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, feed_forward: FeedForward | None = None, ff_norm: Norm | None = None):
+        self.mixer, self.mixer_norm, self.feed_forward, self.ff_norm = mixer, mixer_norm, feed_forward, ff_norm
+
+    def owned_parts(self):
+        return [p for p in (self.mixer, self.mixer_norm, self.feed_forward, self.ff_norm) if p is not None]
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for p in self.owned_parts())
+
+    def first_norm(self):
+        return None  # the stream meets a part first
+
+    def forward(self, resid, pending, ctx, cache, next_norm=None):
+        x = self._read(resid, pending)
+        x = self._take_up(resid, self.mixer.forward(x, ctx, cache), self.mixer_norm)
+        if self.feed_forward is not None:
+            more = {"leave_bias": True} if self.feed_forward.leaves_bias else {}
+            x = self._take_up(resid, self.feed_forward.forward(x, ctx, **more), self.ff_norm)
+        return ops.StreamCopy(x)
+
+    def _read(self, resid, pending):
+        """The stream's rows in the compute type, with everything added."""
+        if isinstance(pending, ops.StreamCopy):
+            return pending.rows
+        delta, alpha = ops.split_pending(pending)
+        if delta is not None:
+            ops.stream_inject(resid, delta, alpha)
+        return resid if self.mixer_norm.out_dtype == torch.float32 else resid.to(self.mixer_norm.out_dtype)
+
+    @staticmethod
+    def _take_up(resid, result, norm):
+        bias = None
+        if isinstance(result, ops.Biased):
+            result, bias = result.tensor, result.bias
+        result, alpha = ops.split_pending(result)
+        if alpha != 1.0:
+            result = result * alpha
+        copy_dtype = norm.out_dtype if norm.out_dtype != torch.float32 else None
+        copy = norm.after_forward(resid, result, bias=bias, copy_dtype=copy_dtype)
+        return resid if copy is None else copy
+
+
+class PostNormMixerOnlyBlock(PostNormBlock):
+    """The same without a feed-forward: ``x <- x + norm1(mixer(x))``."""
+
+    roles = {"mixer": "mixer", "mixer_norm": "norm"}
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm):
+        super().__init__(mixer, mixer_norm)
+
+
 class HyperConnectionBlock(Block):
     """A pre-norm layer over a residual stream kept in S copies ``x_1 .. x_S`` (hyper-connections).  For each of its parts
     q (1: the mixer, 2: the feed-forward) it owns ``hc<q>.in [S]``, ``hc<q>.out [S]`` and ``hc<q>.mix [S, S]``:
@@ -274,5 +338,7 @@ register_part("block", "hyper_connection", HyperConnectionBlock)
 register_part("block", "hyper_connection_mixer_only", HyperConnectionMixerOnlyBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "parallel_mixer_only", ParallelMixerOnlyBlock)
+register_part("block", "post_norm", PostNormBlock)
+register_part("block", "post_norm_mixer_only", PostNormMixerOnlyBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "pre_norm_mixer_only", MixerOnlyBlock)

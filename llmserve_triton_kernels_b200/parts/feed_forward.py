@@ -1,4 +1,4 @@
-"""Dense gated feed-forward: ``down(act(gate(x)) * up(x))`` without biases.
+"""Dense gated feed-forward: ``down(act(gate(x)) * up(x))``, with or without biases.
 
 Parity: src/llmserve/model/llama.py:112-120, where the activation is SiLU
 (``z * sigmoid(z)``); the gate and up matrices are stacked at load so that one matrix product
@@ -12,7 +12,7 @@ import torch
 from .. import ops
 from .base import FeedForward, TensorSpec, register_part
 
-_ACTIVATIONS = ("silu",)
+_ACTIVATIONS = ("silu", "gelu_tanh")
 
 
 class GatedMLP(FeedForward):
@@ -31,7 +31,7 @@ class GatedMLP(FeedForward):
         self.activation = activation
         self.bias = bool(bias)  # ``*_proj.bias`` vectors (none in Llama): products and bias sums as kernels of their own
         self.b_gate_up: torch.Tensor | None = None
-        self.b_down: torch.Tensor | None = None
+        self.b_down_32: torch.Tensor | None = None
         self.w_gate_up: torch.Tensor | None = None  # [2 I, hidden]: gate rows, then up rows
         self.w_down: torch.Tensor | None = None  # [hidden, I]
 
@@ -52,15 +52,20 @@ class GatedMLP(FeedForward):
         self.w_down = tensors[self.names["down"]].to(device=device, dtype=dtype).contiguous()
         if self.bias:
             self.b_gate_up = torch.cat([tensors[self.names["gate_bias"]].to(dtype), tensors[self.names["up_bias"]].to(dtype)]).to(device).contiguous()
-            self.b_down = tensors[self.names["down_bias"]].to(device=device, dtype=dtype).contiguous()
+            self.b_down_32 = tensors[self.names["down_bias"]].to(device=device, dtype=torch.float32).contiguous()  # the sum it joins is 32-bit
 
     accepts_sink = True
 
-    def forward(self, x, ctx, sink=None):
+    @property
+    def leaves_bias(self) -> bool:
+        return self.bias
+
+    def forward(self, x, ctx, sink=None, leave_bias=False):
         if self.bias:
-            act = ops.swiglu(ops.linear(x, self.w_gate_up), self.b_gate_up)  # the bias joins in the activation's kernel
-            return ops.add_bias(ops.linear(act, self.w_down, out_dtype=torch.float32), self.b_down.float())
-        act = ops.linear_swiglu(x, self.w_gate_up)
+            act = ops.swiglu(ops.linear(x, self.w_gate_up), self.b_gate_up, self.activation)  # the bias joins in the activation's kernel
+            out = ops.linear(act, self.w_down, out_dtype=torch.float32)
+            return ops.Biased(out, self.b_down_32) if leave_bias else ops.add_bias(out, self.b_down_32)
+        act = ops.linear_swiglu(x, self.w_gate_up) if self.activation == "silu" else ops.swiglu(ops.linear(x, self.w_gate_up), None, self.activation)
         if sink is not None:
             handed_on = sink.linear(act, self.w_down)
             if handed_on is not None:
@@ -264,15 +269,19 @@ register_part("feed_forward", "table_routed_mlp", TableRoutedMLP)
 
 
 class RoutedGatedMLP(FeedForward):
-    """A mixture of small gated feed-forward layers ``down_e(silu(gate_e x) * up_e x)`` without biases, of which each token
-    uses ``top``, chosen by a router with a bias:
+    """A mixture of small gated feed-forward layers without biases, of which each token uses ``top``, chosen by a router:
 
-        z = W_router x + b_router (32-bit)
-        chosen: the ``top`` experts with the largest z; weights: the softmax over the chosen logits alone
-        out = sum over the chosen e of weight_e * expert_e(x)  +  shared(x)
+        expert(x):  g = min(W_gate x, limit)     u = clamp(W_up x, -limit, limit)
+                    W_down (g * sigmoid(slope * g) * (u + up_shift))        (no limit, slope 1, shift 0: silu(gate) * up)
+        z = W_router x (+ b_router) (32-bit)
+        softmax:  chosen: the ``top`` experts with the largest z; weights: the softmax over the chosen logits alone
+        sigmoid:  s = sigmoid(z); chosen: the ``top`` experts with the largest s + correction; weights: s of the chosen ones over
+                  their sum (+ 1e-20).  With ``groups = (count, keep)`` the experts form ``count`` equal runs of neighbours, a run's
+                  score is the sum of its two largest s + correction, and only experts of the ``keep`` best runs can be chosen
+        out = sum over the chosen e of router_scale * weight_e * expert_e(x)  +  shared(x)
 
-    ``shared_size``: the inner size of an expert of the same form that every token uses with weight one (None: none).
-    Tensors: ``router``, ``router.b``, ``e<i>.gate``, ``e<i>.up``, ``e<i>.down``, ``shared.gate``, ``shared.up``, ``shared.down``.
+    ``shared_size``: the inner size of an expert of the same form that every token uses with weight one (None: none), bounded by
+    ``shared_limit``.  Tensors: ``router``, ``router.b`` (``router_bias``), ``correction`` (``correction``), ``e<i>.gate``, ``e<i>.up``, ``e<i>.down``, ``shared.gate``, ``shared.up``, ``shared.down``.
     As in :class:`TableRoutedMLP` all experts' gate and up matrices are stacked (the shared expert's last) and the down
     matrices stand side by side: a step is one kernel for the router (its 32-bit product, the choice and the weights), one
     product over every expert, one kernel for the activation times the token's weight of each expert's block of columns
@@ -282,12 +291,25 @@ class RoutedGatedMLP(FeedForward):
     accepts_sink = True
     takes_factored = False  # the router reads the normed rows themselves: the norm in front runs as its own kernel
 
-    def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, shared_size: int | None = None, router_bias: bool = True):
+    def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, shared_size: int | None = None, router_bias: bool = True,
+                 scores: str = "softmax", correction: bool = False, groups: tuple[int, int] | None = None, router_scale: float = 1.0,
+                 limit: float | None = None, shared_limit: float | None = None, slope: float = 1.0, up_shift: float = 0.0):
         if not 1 <= int(top) <= int(experts):
             raise ValueError(f"a token uses {top} of {experts} experts")
         self.hidden_size, self.experts, self.top, self.expert_size = int(hidden_size), int(experts), int(top), int(expert_size)
         self.shared_size = int(shared_size) if shared_size else 0
         self.router_bias = bool(router_bias)
+        if scores not in ("softmax", "sigmoid") or (scores == "softmax" and (correction or groups)):
+            raise ValueError(f"router scores are 'softmax', or 'sigmoid' with a correction and groups if there are any; got {scores!r}")
+        self.scores, self.has_correction, self.router_scale = scores, bool(correction), float(router_scale)
+        self.groups = None if groups is None else (int(groups[0]), int(groups[1]))
+        if self.groups and not (1 <= self.groups[1] <= self.groups[0] and self.experts % self.groups[0] == 0
+                                and self.top <= self.groups[1] * (self.experts // self.groups[0])):
+            raise ValueError(f"{self.top} of {self.experts} experts cannot be chosen from {self.groups[1]} of {self.groups[0]} equal groups")
+        self.limit = float("inf") if limit is None else float(limit)
+        self.shared_limit = self.limit if shared_limit is None else float(shared_limit)
+        self.slope, self.up_shift = float(slope), float(up_shift)
+        self.correction: torch.Tensor | None = None
         self.w_router = self.b_router = self.w_up = self.w_down = None
 
     def tensors(self) -> dict[str, TensorSpec]:
@@ -295,6 +317,8 @@ class RoutedGatedMLP(FeedForward):
         specs = {"router": TensorSpec((self.experts, h))}
         if self.router_bias:
             specs["router.b"] = TensorSpec((self.experts,))
+        if self.has_correction:
+            specs["correction"] = TensorSpec((self.experts,))
         for e in range(self.experts):
             specs[f"e{e}.gate"] = TensorSpec((f, h))
             specs[f"e{e}.up"] = TensorSpec((f, h))
@@ -313,12 +337,15 @@ class RoutedGatedMLP(FeedForward):
         self.w_router = tensors["router"].to(device=device, dtype=torch.float32).contiguous()
         if self.router_bias:
             self.b_router = tensors["router.b"].to(device=device, dtype=torch.float32).contiguous()
+        if self.has_correction:
+            self.correction = tensors["correction"].to(device=device, dtype=torch.float32).contiguous()
 
     def forward(self, x, ctx, sink=None):
         xt = x.materialize() if isinstance(x, ops.NormedInput) else x
-        weights = ops.route(xt, self.w_router, None, self.experts, self.top, 1.0, True, False, bias=self.b_router, shared_one=self.shared_size > 0)
-        act = ops.expert_gated_act(ops.linear(xt, self.w_up), self.experts, self.expert_size, self.shared_size, float("inf"), float("inf"), 1.0,
-                                   weights=weights, up_shift=0.0)
+        weights = ops.route(xt, self.w_router, self.correction, self.experts, self.top, self.router_scale, True, False, bias=self.b_router,
+                            shared_one=self.shared_size > 0, scores=self.scores, groups=self.groups)
+        act = ops.expert_gated_act(ops.linear(xt, self.w_up), self.experts, self.expert_size, self.shared_size, self.limit, self.shared_limit,
+                                   self.slope, weights=weights, up_shift=self.up_shift)
         if sink is not None:
             handed_on = sink.linear(act, self.w_down)
             if handed_on is not None:

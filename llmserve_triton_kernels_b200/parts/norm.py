@@ -1,4 +1,4 @@
-"""RMS normalisation with the residual sum fused in.
+"""RMS normalisation with the residual sum fused in, and layer normalisation.
 
 Parity: src/llmserve/model/llama.py:18-28 — mean of squares, ``+ eps`` and rsqrt in 32-bit,
 then the weight multiply.  Here the residual stream itself is 32-bit and the result is rounded
@@ -69,6 +69,12 @@ class RMSNorm(Norm):
             raise NotImplementedError("a norm in groups behind a stream kept in copies is not built")
         return ops.hyper_mix_norm(streams, update, read_in, self.weight, self.eps, rows=rows, out_dtype=self.out_dtype)
 
+    def after_forward(self, resid, result, bias=None, copy_dtype=None):
+        """``resid += norm(result + bias)`` in place: this norm behind a part (see ``ops.post_norm_add``)."""
+        if self.groups != 1:
+            raise NotImplementedError("a norm in groups behind a part is not built")
+        return ops.post_norm_add(resid, result, self.weight, self.eps, bias=bias, copy_dtype=copy_dtype, center=False)
+
     def add_forward(self, resid, delta, rows=None, alpha: float = 1.0):
         if self.groups == 1 and alpha == 1.0:
             return ops.rmsnorm(resid, self.weight, self.eps, delta=delta, rows=rows, out_dtype=self.out_dtype)
@@ -76,3 +82,36 @@ class RMSNorm(Norm):
 
 
 register_part("norm", "rms_norm", RMSNorm)
+
+
+class LayerNorm(Norm):
+    """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight`` over the row, without a bias; statistics in 32-bit.  ``weight_name``
+    as in :class:`RMSNorm`."""
+
+    graph_safe = True
+
+    def __init__(self, size: int, eps: float, weight_name: str = "weight"):
+        self.size, self.eps, self.weight_name = int(size), float(eps), weight_name
+        self.weight: torch.Tensor | None = None
+        self.out_dtype: torch.dtype | None = None
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        return {self.weight_name: TensorSpec((self.size,), init="ones_plus_normal")}
+
+    def bind(self, tensors, dtype, device) -> None:
+        self.weight = tensors[self.weight_name].to(device=device, dtype=torch.float32).contiguous()
+        self.out_dtype = dtype
+
+    def forward(self, x, rows=None):
+        return self.add_forward(x, None, rows)
+
+    def add_forward(self, resid, delta, rows=None, alpha: float = 1.0):
+        delta = delta if delta is None or delta.dtype == torch.float32 else delta.float()
+        return ops.layer_norm(resid, self.weight, self.eps, delta=delta, alpha=alpha, rows=rows, out_dtype=self.out_dtype)
+
+    def after_forward(self, resid, result, bias=None, copy_dtype=None):
+        """``resid += norm(result + bias)`` in place: this norm behind a part (see ``ops.post_norm_add``)."""
+        return ops.post_norm_add(resid, result, self.weight, self.eps, bias=bias, copy_dtype=copy_dtype)
+
+
+register_part("norm", "layer_norm", LayerNorm)

@@ -1,6 +1,6 @@
 """Recurrences with a fixed-size state per request: an element-wise gated one (minGRU), one whose state is a matrix per
-head that decays by a fixed factor (retention), and one whose matrix decays row by row as each token chooses (gated linear
-attention).
+head that decays by a fixed factor (retention), one whose matrix decays row by row as each token chooses (gated linear
+attention), and one whose matrix is corrected towards each token's value at its key (the gated delta rule).
 
 minGRU: the update gate and the candidate read only the current token,
 
@@ -17,7 +17,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import Mixer, StateSpec, TensorSpec, register_part
+from .base import CompositeSpec, Mixer, StateSpec, TensorSpec, register_part
 
 _NAMES = {"z": "z", "z_bias": "z.b", "x": "x", "x_bias": "x.b", "gate": "g", "out": "o"}
 
@@ -208,3 +208,97 @@ class GatedLinearAttention(Mixer):
 
 
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
+
+
+class GatedDeltaRule(Mixer):
+    """Linear attention whose state forgets by a factor of the token's choosing and is corrected, not only added to:
+
+        q = W_q x, k = W_k x (kv_heads x dim), v = W_v x (heads x value_dim), g = W_g x
+        q, k, v: every channel through a short causal convolution over time (weights ``<name>.conv`` [channels, taps]), then silu
+        q, k: unit vectors per head, y / sqrt(sum y^2 + 1e-6); q then times dim^(-1/2); head h reads q/k head h // (heads / kv_heads)
+        beta = sigmoid(W_b x)        a = exp(-exp(A_log) * softplus(W_a x + dt_bias))                  (one number a head each)
+        S <- a S        u = beta (v - S^T k)        S <- S + k u^T        o = S^T q                     per head
+        out = W_o (rmsnorm_per_head(o) * w_norm * silu(g))                                             (w_norm [value_dim], shared)
+
+    S ``[heads, dim, value_dim]`` starts at zero, is 32-bit and lives in the request's slot of the cache manager; so do the
+    convolutions' last ``taps - 1`` input rows.  The six input projections are one stacked product whose result stays 32-bit, so
+    that everything that enters the recurrence is."""
+
+    graph_safe = True
+    accepts_sink = True
+    takes_projection = True  # a mixer that runs this one beside others may run the input product itself (``forward(proj=)``)
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, conv: int, norm_eps: float,
+                 tensor_names: dict[str, str] | None = None):
+        if num_heads % num_kv_heads:
+            raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
+        if not 1 <= int(head_dim) <= 256:
+            raise ValueError(f"head_dim {head_dim}: the recurrence's kernel takes keys of up to 256 lanes")
+        if not 1 <= int(conv) <= 16:
+            raise ValueError(f"a short convolution has 1 to 16 taps, got {conv}")
+        self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.head_dim, self.value_dim, self.conv, self.norm_eps = int(head_dim), int(value_dim), int(conv), float(norm_eps)
+        self.names = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o", "beta": "b", "decay": "a", "a_log": "A_log", "dt_bias": "dt_bias",
+                      "norm": "norm", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", **(tensor_names or {})}
+        self.w_in = self.w_out = self.w_conv = self.a_log = self.dt_bias = self.norm_weight = None
+        self.dtype: torch.dtype | None = None
+
+    def _rows(self) -> dict[str, int]:
+        """Rows of the stacked input product by role, in the order of its columns."""
+        qk, vv = self.num_kv_heads * self.head_dim, self.num_heads * self.value_dim
+        return {"q": qk, "k": qk, "v": vv, "gate": vv, "beta": self.num_heads, "decay": self.num_heads}
+
+    def tensors(self) -> dict[str, TensorSpec]:
+        n, h, rows = self.names, self.hidden_size, self._rows()
+        specs = {n[role]: TensorSpec((count, h)) for role, count in rows.items()}
+        specs[n["out"]] = TensorSpec((h, self.num_heads * self.value_dim))
+        for role in ("q", "k", "v"):
+            specs[n[role + "_conv"]] = TensorSpec((rows[role], self.conv), init="mean_plus_normal")
+        for role in ("a_log", "dt_bias"):
+            specs[n[role]] = TensorSpec((self.num_heads,))
+        specs[n["norm"]] = TensorSpec((self.value_dim,), init="ones_plus_normal")
+        return specs
+
+    def bind(self, tensors, dtype, device) -> None:
+        n = self.names
+        mats = [tensors[n[role]].to(dtype) for role in self._rows()]
+        rows = sum(m.shape[0] for m in mats)
+        if rows % 16:  # a few rows of zeros, so that the stacked product's rows stay on wide boundaries
+            mats.append(torch.zeros((16 - rows % 16, self.hidden_size), dtype=dtype, device=mats[0].device))
+        self.w_in = torch.cat(mats, dim=0).to(device).contiguous()
+        self.w_out = tensors[n["out"]].to(device=device, dtype=dtype).contiguous()
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()  # noqa: E731
+        self.w_conv = f32(torch.cat([tensors[n[r + "_conv"]].float() for r in ("q", "k", "v")], dim=0))
+        self.a_log, self.dt_bias, self.norm_weight = f32(tensors[n["a_log"]]), f32(tensors[n["dt_bias"]]), f32(tensors[n["norm"]])
+        self.dtype = dtype
+
+    def cache_spec(self):
+        state = StateSpec((self.num_heads, self.head_dim, self.value_dim), torch.float32)
+        if self.conv == 1:
+            return state
+        return CompositeSpec((state, StateSpec((self.conv - 1, self.conv_channels), torch.float32)))
+
+    @property
+    def conv_channels(self) -> int:
+        rows = self._rows()
+        return rows["q"] + rows["k"] + rows["v"]
+
+    def forward(self, x, ctx, cache, sink=None, proj=None):
+        H, V, C = self.num_heads, self.value_dim, self.conv_channels
+        if proj is None:
+            proj = ops.linear(x, self.w_in, out_dtype=torch.float32)  # [N, q | k | v | gate | beta | decay], 32-bit
+        state, tail = (cache, None) if self.conv == 1 else cache.parts
+        y = ops.short_conv(proj, self.w_conv, None if tail is None else tail.states, state.slots if tail is None else tail.slots, ctx,
+                           channels=C, activation="silu")
+        b = C + H * V
+        out = ops.delta_rule(y, proj[:, b : b + H], proj[:, b + H : b + 2 * H], self.a_log, self.dt_bias, proj[:, C:b], self.norm_weight, self.norm_eps,
+                             state.states, state.slots, ctx, heads=H, kv_heads=self.num_kv_heads, dim=self.head_dim, value_dim=V,
+                             out_dtype=self.dtype)
+        if sink is not None:
+            handed_on = sink.linear(out, self.w_out)
+            if handed_on is not None:
+                return handed_on
+        return ops.linear(out, self.w_out, out_dtype=torch.float32)
+
+
+register_part("mixer", "gated_delta_rule", GatedDeltaRule)

@@ -94,11 +94,17 @@ def paged_attention(qkv, pool, page_table, ctx, *, num_heads, num_kv_heads, head
     return out
 
 
-def swiglu(gate_up, bias=None):
+def embed_positions(ids, table, positions, pos, scale=1.0, copy_dtype=None):
+    x = table[ids.long()].float() * scale + pos[positions.long()].float()
+    return x, None if copy_dtype is None else x.to(copy_dtype)
+
+
+def swiglu(gate_up, bias=None, activation="silu"):
     inter = gate_up.shape[1] // 2
     row = gate_up.float() if bias is None else gate_up.float() + bias.float()
     g, u = row[:, :inter], row[:, inter:]
-    return (g * torch.sigmoid(g) * u).to(gate_up.dtype)
+    act = unary(g, "gelu_tanh") if activation == "gelu_tanh" else g * torch.sigmoid(g)
+    return (act * u).to(gate_up.dtype)
 
 
 def add_bias(x, bias):
@@ -166,6 +172,8 @@ def unary(x, kind, alpha=1.0, inplace=False, out=None):
         y = alpha * v
     elif kind == "silu":
         y = v * torch.sigmoid(v)
+    elif kind == "softcap":
+        y = alpha * torch.tanh(v / alpha)
     else:
         raise ValueError(kind)
     if inplace:
@@ -608,7 +616,28 @@ def route_topk(z, correction, experts, top, scale=1.0, renormalize=False, shared
     return w
 
 
-def route(x, w_router, correction, experts, top, scale=1.0, renormalize=False, shared_gate=False, bias=None, shared_one=False):
+def _route_sigmoid(z, correction, experts, top, scale, groups):
+    s = torch.sigmoid(z[:, :experts])
+    choice = s if correction is None else s + correction.float()
+    if groups is not None:
+        count, keep = groups
+        each = choice.view(choice.shape[0], count, -1)
+        score = each.sort(dim=-1, descending=True).values[..., :2].sum(-1)
+        best = score.sort(dim=-1, descending=True, stable=True).indices[:, :keep]  # the lowest index among equals, as the kernel
+        stays = torch.zeros_like(score, dtype=torch.bool).scatter_(1, best, True)
+        choice = choice.masked_fill(~stays.repeat_interleave(each.shape[2], dim=1), float("-inf"))
+    chosen = torch.zeros_like(s).scatter_(1, choice.sort(dim=-1, descending=True, stable=True).indices[:, :top], 1.0)
+    w = s * chosen
+    return w / (w.sum(-1, keepdim=True) + 1e-20) * scale
+
+
+def route(x, w_router, correction, experts, top, scale=1.0, renormalize=False, shared_gate=False, bias=None, shared_one=False, scores="softmax",
+          groups=None):
+    if scores == "sigmoid":
+        assert renormalize and not shared_gate and bias is None
+        w = _route_sigmoid(x.float() @ w_router.float().t(), correction, experts, top, scale, groups)
+        return torch.cat((w, torch.ones_like(w[:, :1])), dim=1) if shared_one else w
+    assert groups is None
     z = x.float() @ w_router.float().t()
     if bias is not None:
         z = torch.cat((z[:, :experts] + bias.float(), z[:, experts:]), dim=1)
@@ -616,7 +645,7 @@ def route(x, w_router, correction, experts, top, scale=1.0, renormalize=False, s
     return torch.cat((w, torch.ones_like(w[:, :1])), dim=1) if shared_one else w
 
 
-def short_conv(u, weight, states, state_slots, ctx, channels=None):
+def short_conv(u, weight, states, state_slots, ctx, channels=None, activation=None):
     c = int(channels) if channels is not None else weight.shape[0]
     taps = weight.shape[1]
     out = torch.empty((u.shape[0], c), dtype=torch.float32, device=u.device)
@@ -628,7 +657,48 @@ def short_conv(u, weight, states, state_slots, ctx, channels=None):
             rows = torch.cat((states[slots[r]], rows), dim=0)
             states[slots[r]] = rows[rows.shape[0] - (taps - 1) :]
         out[t0:t1] = sum(weight[:, j].float()[None, :] * rows[j : j + (t1 - t0)] for j in range(taps))
-    return out
+    return out * torch.sigmoid(out) if activation == "silu" else out
+
+
+def layer_norm(x, weight, eps, delta=None, alpha=1.0, rows=None, out_dtype=torch.float32, center=True):
+    if rows is not None:
+        v = x[rows.long()] if delta is None else x[rows.long()] + alpha * delta[rows.long()]
+    else:
+        if delta is not None:
+            x.add_(delta, alpha=alpha)
+        v = x
+    return _normed(v, weight, eps, center).to(out_dtype)
+
+
+def _normed(v, weight, eps, center):
+    v = v - v.mean(-1, keepdim=True) if center else v
+    return v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight
+
+
+def post_norm_add(stream, y, weight, eps, bias=None, copy_dtype=None, center=True):
+    stream.add_(_normed(y if bias is None else y + bias, weight, eps, center))
+    return None if copy_dtype is None else stream.to(copy_dtype)
+
+
+def delta_rule(y, beta, decay, a_log, dt_bias, gate, weight, eps, states, state_slots, ctx, *, heads, kv_heads, dim, value_dim, out_dtype):
+    n, qk, rep = y.shape[0], kv_heads * dim, heads // kv_heads
+    unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)  # noqa: E731
+    q = unit(y[:, :qk].reshape(n, kv_heads, dim)).repeat_interleave(rep, dim=1) * dim ** -0.5
+    k = unit(y[:, qk : 2 * qk].reshape(n, kv_heads, dim)).repeat_interleave(rep, dim=1)
+    v = y[:, 2 * qk : 2 * qk + heads * value_dim].reshape(n, heads, value_dim)
+    b = torch.sigmoid(beta[:, :heads])
+    g = torch.exp(-torch.exp(a_log) * torch.nn.functional.softplus(decay[:, :heads] + dt_bias, threshold=60.0))
+    o = torch.empty((n, heads, value_dim), dtype=torch.float32, device=y.device)
+    cu, slots = ctx.cu_tokens.tolist(), state_slots.tolist()
+    for r in range(len(cu) - 1):
+        S = states[slots[r]].clone()
+        for t in range(cu[r], cu[r + 1]):
+            S = S * g[t][:, None, None]
+            u = b[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        states[slots[r]] = S
+    return head_norm_gate(o, gate[:, : heads * value_dim], eps, "silu", out_dtype=out_dtype, weight=weight)
 
 
 def row_rmsnorm(x, weight, eps, out_dtype=None):
@@ -656,6 +726,10 @@ def branch_sum_rmsnorm(pending, resid, weight, eps, out_dtype):
 
 
 ALL = (
+    "embed_positions",
+    "layer_norm",
+    "post_norm_add",
+    "delta_rule",
     "shift_norm",
     "short_conv",
     "row_rmsnorm",
