@@ -14,7 +14,7 @@ cache of the live requests) to its time; ``points`` holds decode at batch 1 and 
 Peaks come from MEASURED_PEAKS.json beside this file when present, else from an earlier
 measurement on the same pool (and the line says which).
 
-``python bench.py --design nurolorn-small|nurolorn-1b|kafepel-small|kafepel-1b|nudodra-small|nudodra-1b|tenotar-small|tenotar-1b|pefedra-small|pefedra-1b`` prints, instead of the line, prefill and decode
+``python bench.py --design nurolorn-small|nurolorn-1b|kafepel-small|kafepel-1b|nudodra-small|nudodra-1b|tenotar-small|tenotar-1b|pefedra-small|pefedra-1b|zifuzen-small|zifuzen-1b`` prints, instead of the line, prefill and decode
 throughput of that configuration beside a Llama of equal width, depth and feed-forward size, and the design's kernels against
 their rooflines.
 
@@ -221,12 +221,13 @@ def design_comparison(args) -> int:
     nudodra = design["architecture"] == "Nudodra"
     tenotar = design["architecture"] == "Tenotar"
     pefedra = design["architecture"] == "Pefedra"
-    if nudodra or tenotar:  # no dense feed-forward (or one layer's only): the twin's has the size of what a token uses (its chosen experts and the shared one)
+    zifuzen = design["architecture"] == "Zifuzen"
+    if nudodra or tenotar or zifuzen:  # no dense feed-forward (or one layer's only): the twin's has the size of what a token uses (its chosen experts and the shared one)
         moe = next(x["mlp"] for x in design["layers"] if x.get("mlp") and x["mlp"].get("kind", "moe") == "moe")
         ff = moe["router"]["top"] * moe["expert"]["ff"] + (moe["shared"]["ff"] if moe.get("shared") else 0)
     else:
         ff = next(x["mlp"]["ff"] for x in design["layers"] if x.get("mlp") and "ff" in x["mlp"])
-    gated = design["architecture"] in ("Kafepel", "Nudodra", "Tenotar")  # their feed-forwards have three matrices, like the twin's
+    gated = design["architecture"] in ("Kafepel", "Nudodra", "Tenotar", "Zifuzen")  # their feed-forwards have three matrices, like the twin's
     twin = {
         "architectures": ["LlamaForCausalLM"], "model_type": "llama", "hidden_act": "silu", "rope_theta": 10000.0, "rms_norm_eps": 1e-5,
         "tie_word_embeddings": False, "vocab_size": vocab, "hidden_size": width, "intermediate_size": ff if gated else (ff * 2 // 3 + 63) // 64 * 64,
@@ -269,6 +270,8 @@ def design_comparison(args) -> int:
         compared.insert(1, ("tenotar-twin", {
             "architecture": "Tenotar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
             "layers": [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": twin["intermediate_size"]}} for _ in design["layers"]]}))
+    if zifuzen:  # the closest design the engine has: a gated recurrence and softmax attention with shared pages, bounded gated experts, at the same sizes
+        compared.insert(1, (args.design.replace("zifuzen", "nudodra"), dict(PRESETS[args.design.replace("zifuzen", "nudodra")])))
     for name, cfg_dict in compared:
         a = architecture_of(cfg_dict)
         model = random_model(a.config_class.from_dict(cfg_dict), 0, "bfloat16", device)
@@ -341,8 +344,8 @@ def design_comparison(args) -> int:
 
     bf = torch.bfloat16
     kernels = {}
-    if design["architecture"] in ("Kafepel", "Nudodra", "Tenotar", "Pefedra"):
-        (_pefedra_kernels if pefedra else _tenotar_kernels if tenotar else _nudodra_kernels if nudodra else _kafepel_kernels)(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device)
+    if design["architecture"] in ("Kafepel", "Nudodra", "Tenotar", "Pefedra", "Zifuzen"):
+        (_zifuzen_kernels if zifuzen else _pefedra_kernels if pefedra else _tenotar_kernels if tenotar else _nudodra_kernels if nudodra else _kafepel_kernels)(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device)
         out["kernels"] = kernels
         out["peaks"] = {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"]}
         print(json.dumps(out, indent=1))
@@ -678,6 +681,108 @@ def _tenotar_kernels(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor,
         hbm(f"nudodra_expert_gated_act_{label}", us, n * ((top * eff + sff) * 4 + (E * eff + sff) * 2))
 
 
+def _zifuzen_kernels(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device) -> None:
+    """The Zifuzen design's own kernels, alone, at the preset's sizes: one request of 2,048 prompt tokens, and 8 decoding requests of
+    2,048 cached tokens; beside each the like kernel of the Nudodra design (the closest one the engine has), or of the design that
+    has one, at the same sizes."""
+    bf = torch.bfloat16
+    R, A = (next(x["mixer"] for x in design["layers"] if x["type"] == kind) for kind in ("delta", "attention"))
+    moe = next(x["mlp"] for x in design["layers"] if x["mlp"] and x["mlp"]["kind"] == "moe")
+    dense_ff = next(x["mlp"]["ff"] for x in design["layers"] if x["mlp"] and x["mlp"]["kind"] == "dense")
+    width = design["width"]
+    H, KV, D, V = A["heads"], A["kv_heads"], A["dim"], A["vdim"]
+    RH, RG, RD, RV = R["heads"], R["kv_heads"], R["dim"], R["vdim"]
+    for label, qs, cs in (("prefill_2048", [2048], [2048]), ("decode_8x2048", [1] * 8, [2048] * 8)):
+        ctx, table, slots, pages = ctx_for(qs, cs)
+        n = ctx.num_tokens
+        pairs = sum(q * c - q * (q - 1) // 2 for q, c in zip(qs, cs))
+        prefill = label.startswith("prefill")
+        sl = i32(list(range(len(qs))))
+        # the recurrence with its step sizes, decays, unit vectors, head norm and gate, beside Nudodra's scan and head norm
+        C = 2 * RG * RD + RH * RV
+        y, proj = torch.randn(n, C, device=device), torch.randn(n, RH * RV + 2 * RH, device=device)
+        states = torch.zeros(8, RH, RD, RV, device=device)
+        a_log, dt, wn = torch.zeros(RH, device=device), torch.full((RH,), -2.0, device=device), torch.ones(RV, device=device)
+        state_bytes = 2 * len(qs) * RH * RD * RV * 4
+        us = timed(lambda: ops.delta_rule(y, proj[:, RH * RV : RH * RV + RH], proj[:, RH * RV + RH :], a_log, dt, proj[:, : RH * RV], wn, 1e-6, states, sl,
+                                          ctx, heads=RH, kv_heads=RG, dim=RD, value_dim=RV, out_dtype=bf))
+        hbm(f"delta_rule_with_norm_and_gate_{label}", us, n * (2 * RG * RD + RH * (2 * RV + 2)) * 4 + n * RH * RV * 2 + state_bytes, like="gated_scan + head_norm_gate")
+        rq, rk, rz = (torch.randn(n, RH * RD, device=device) for _ in range(3))
+        rv, zb = torch.randn(n, RH * RV, device=device), torch.full((RH * RD,), 3.0, device=device)
+
+        def nudodra_scan():
+            o = ops.gated_scan(rq, rk, rv, rz, zb, 0.125, RD ** -0.5, states, sl, ctx.cu_tokens, len(qs), RH, RD, RV, max(qs))
+            ops.head_norm_gate(o, proj[:, : RH * RV], 1e-6, "silu", bf, weight=wn)
+
+        us = timed(nudodra_scan)
+        hbm(f"nudodra_gated_scan_with_norm_and_gate_{label}", us, n * RH * (3 * RD + 2 * RV) * 4 + n * RH * RV * 2 + state_bytes)
+        # the convolution with silu behind it beside Tenotar's without
+        u, w = torch.randn(n, C, device=device), torch.randn(C, R["conv"], device=device)
+        rows = torch.zeros(8, R["conv"] - 1, C, device=device)
+        for name, act in (("short_conv_silu", "silu"), ("tenotar_short_conv", None)):
+            us = timed(lambda: ops.short_conv(u, w, rows, sl, ctx, activation=act))
+            hbm(f"{name}_{label}", us, n * C * 8, like="short_conv" if act else None)
+        # the norm behind a part with the sum and the copy beside the norm in front of one with the sum
+        stream, delta, part = (torch.randn(n, width, device=device) for _ in range(3))
+        wd = torch.ones(width, device=device)
+        us = timed(lambda: ops.post_norm_add(stream, part, wd, 1e-6, copy_dtype=bf))
+        hbm(f"post_norm_add_{label}", us, n * width * 14, like="rmsnorm with the sum")
+        us = timed(lambda: ops.rmsnorm(stream, wd, 1e-6, delta=delta, out_dtype=bf))
+        hbm(f"llama_rmsnorm_with_sum_{label}", us, n * width * 14)
+        # attention over all keys, and the heads' preparation
+        pool = torch.randn(pages, 2, KV, 16, max(D, V), device=device).to(bf)
+        q = (torch.randn(n, H * D, device=device) * 0.3).to(bf)
+        kw = dict(num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=V, scale=A["scale"])
+        work = 2.0 * pairs * H * (D + V) if prefill else sum(cs) * KV * (D + V) * 2 + n * H * (D + V) * 2
+        us = timed(lambda: ops.paged_softmax_attention(q, pool, table, ctx, **kw))
+        (tensor if prefill else hbm)(f"attention_{label}", us, work, like="sink_attention")
+        sinks = torch.zeros(H, device=device)
+        us = timed(lambda: ops.paged_softmax_attention(q, pool, table, ctx, **kw, sinks=sinks))
+        (tensor if prefill else hbm)(f"nudodra_sink_attention_{label}", us, work)
+        hp, qw, kw_ = torch.randn(n, (H + KV) * D + KV * V, device=device), torch.ones(D, device=device), torch.ones(D, device=device)
+        head_bytes = n * ((H + KV) * D + KV * V) * 6
+        us = timed(lambda: ops.head_prepare(hp, ctx.positions, heads=H, kv_heads=KV, dim=D, value_dim=V, q_weight=qw, k_weight=kw_, eps=1e-6, pool=pool, slot_map=slots))
+        hbm(f"head_prepare_{label}", us, head_bytes, like="head_prepare with rotation and biases")
+        freq, b_in = torch.rand(D // 4, device=device), torch.randn((H + KV) * D + KV * V, device=device)
+        us = timed(lambda: ops.head_prepare(hp, ctx.positions, heads=H, kv_heads=KV, dim=D, value_dim=V, bias=b_in, q_weight=qw, k_weight=kw_, eps=1e-6,
+                                            freq=freq, pool=pool, slot_map=slots))
+        hbm(f"nudodra_head_prepare_{label}", us, head_bytes)
+        # the router with sigmoid scores and groups, the experts' activation, the dense layer's
+        E, top, eff, sff = moe["router"]["experts"], moe["router"]["top"], moe["expert"]["ff"], moe["shared"]["ff"]
+        xb, wr, corr = torch.randn(n, width, device=device).to(bf), torch.randn(E, width, device=device) * 0.02, torch.randn(E, device=device)
+        groups = moe["router"]["groups"]
+        router_bytes = n * width * 2 + E * width * 4 + n * (E + 1) * 4
+        us = timed(lambda: ops.route(xb, wr, corr, E, top, 2.5, True, False, shared_one=True, scores="sigmoid", groups=(groups["count"], groups["keep"])))
+        hbm(f"router_with_groups_{label}", us, router_bytes, like="router (the Tenotar design's)")
+        us = timed(lambda: ops.route(xb, wr, None, E, top, 1.0, True, False, bias=corr, shared_one=True))
+        hbm(f"tenotar_router_{label}", us, router_bytes)
+        up2 = torch.randn(n, 2 * (E * eff + sff), device=device).to(bf)
+        wts = ops.route(xb, wr, corr, E, top, 2.5, True, False, shared_one=True, scores="sigmoid", groups=(groups["count"], groups["keep"]))
+        act_bytes = n * ((top * eff + sff) * 4 + (E * eff + sff) * 2)
+        us = timed(lambda: ops.expert_gated_act(up2, E, eff, sff, 7.0, 7.0, 1.702, weights=wts))
+        hbm(f"expert_gated_act_{label}", us, act_bytes, like="expert_gated_act with the table's weights")
+        tab = torch.rand(design["vocab"], E, device=device).argsort(dim=1)[:, :top].to(torch.int32).contiguous()
+        ids = torch.randint(0, design["vocab"], (n,), device=device, dtype=torch.int32)
+        us = timed(lambda: ops.expert_gated_act(up2, E, eff, sff, 7.0, 7.0, 1.702, ids=ids, table=tab))
+        hbm(f"nudodra_expert_gated_act_{label}", us, act_bytes)
+        gu, gb = torch.randn(n, 2 * dense_ff, device=device).to(bf), torch.randn(2 * dense_ff, device=device).to(bf)
+        for name, act in (("gelu_gate", "gelu_tanh"), ("tenotar_silu_gate", "silu")):
+            us = timed(lambda: ops.swiglu(gu, gb, act))
+            hbm(f"{name}_{label}", us, n * dense_ff * 6, like="swiglu with biases" if act != "silu" else None)
+        # the embedding with positions, the logits' cap
+        emb, pos = torch.randn(design["vocab"], width, device=device).to(bf), torch.randn(design["max_positions"], width, device=device).to(bf)
+        us = timed(lambda: ops.embed_positions(ids, emb, ctx.positions, pos, 2.0, copy_dtype=bf))
+        hbm(f"embed_positions_{label}", us, n * width * 10, like="embed")
+        us = timed(lambda: ops.embed(ids, emb))
+        hbm(f"llama_embed_{label}", us, n * width * 6)
+        if not prefill:
+            z = torch.randn(n, design["vocab"], device=device)
+            us = timed(lambda: ops.unary(z, "softcap", 30.0, inplace=True))
+            hbm(f"logit_cap_{label}", us, n * design["vocab"] * 8, like="logit scale")
+            us = timed(lambda: ops.unary(z, "scale", 1.5, inplace=True))
+            hbm(f"logit_scale_{label}", us, n * design["vocab"] * 8)
+
+
 def _pefedra_kernels(design, twin, ops, torch, timed, ctx_for, i32, hbm, tensor, device) -> None:
     """The Pefedra design's own kernels, alone, at the preset's sizes: one request of 2,048 prompt tokens, and 8 decoding requests of
     2,048 cached tokens; beside each the like kernel of the Tenotar design (the closest one the engine has) at the same sizes.
@@ -781,8 +886,8 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers than the configuration has (recorded in config)")
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64, the end-to-end run and the kernel table")
     ap.add_argument("--design", choices=["nurolorn-small", "nurolorn-1b", "kafepel-small", "kafepel-1b", "nudodra-small", "nudodra-1b", "tenotar-small",
-                                         "tenotar-1b", "pefedra-small", "pefedra-1b"], default=None,
-                    help="instead of the one line: prefill and decode throughput of a Nurolorn, Kafepel, Nudodra, Tenotar or Pefedra configuration beside a Llama of "
+                                         "tenotar-1b", "pefedra-small", "pefedra-1b", "zifuzen-small", "zifuzen-1b"], default=None,
+                    help="instead of the one line: prefill and decode throughput of a Nurolorn, Kafepel, Nudodra, Tenotar, Pefedra or Zifuzen configuration beside a Llama of "
                          "equal width, depth and feed-forward size, and the design's own kernels against their rooflines")
     ap.add_argument("--sweep", action="store_true",
                     help="instead of the one line: a table of decode steps over batch sizes and context lengths and of prefills over prompt lengths")

@@ -110,7 +110,33 @@ def _pefedra(width: int, pattern: str, heads: int, kv_heads: int, ff: int, span:
     return {"architecture": "Pefedra", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "layers": layers, "norm": {"eps": 1e-6}}
 
 
+def _zifuzen(width: int, pattern: str, heads: int, kv_heads: int, dense_ff: int, experts: int, top: int, expert_ff: int, shared_ff: int,
+             places: int = 8192, vocab: int = 32000) -> dict:
+    """``pattern``: one letter a layer, D the delta rule with two heads a key head, E with one and shorter values, A attention with
+    pages of its own, a attention that reads the pages of the last A in front of it.  Attention heads of 64 lanes; half as many
+    recurrent heads with keys of 64 and values of 128 (E: 64) lanes behind convolutions of 4 taps; the first layer's feed-forward is
+    dense, the others' a mixture of experts in four groups of which a token uses two."""
+    head, r = 64, heads // 2
+    kinds = {
+        "D": {"type": "delta", "mixer": {"heads": r, "kv_heads": r // 2, "dim": head, "vdim": 2 * head, "conv": 4}},
+        "E": {"type": "delta_2", "mixer": {"heads": r, "kv_heads": r, "dim": head, "vdim": head, "conv": 4}},
+    }
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": expert_ff, "limit": 7.0}, "shared": {"ff": shared_ff, "limit": 7.0}}
+    layers, last = [], None
+    for i, c in enumerate(pattern):
+        kind = kinds.get(c) or {"type": "attention", "mixer": dict(attention) if c == "A" else {**attention, "kv_from": last}}
+        last = i if c == "A" else last
+        layers.append({**kind, "mlp": {"kind": "dense", "ff": dense_ff} if i == 0 else moe})
+    return {"architecture": "Zifuzen", "vocab": vocab, "width": width, "embedding": {"scale": float(width) ** 0.5}, "layers": layers,
+            "norm": {"eps": 1e-6}, "max_positions": places, "logit_softcap": 30.0}
+
+
 PRESETS: dict[str, dict] = {
+    # Zifuzen at the sizes of the Nudodra presets below (the design has no published sizes)
+    "zifuzen-small": _zifuzen(1024, "DEAaDEAa", 16, 4, 2816, 16, 2, 512, 1024),
+    "zifuzen-1b": _zifuzen(2048, "DEAaDEAaDEAa", 32, 8, 5632, 32, 4, 704, 1408),
     # Pefedra at the width and depth of the Tenotar presets below (the design has no published sizes)
     "pefedra-small": _pefedra(1024, "DTTDTTDT", 16, 4, 4096),
     "pefedra-1b": _pefedra(2048, "DTTDTTDTTDTT", 32, 8, 8192),

@@ -22,14 +22,16 @@
 // The first line is a triangular system (I + A) u = beta (v - G S^T k) whose matrix does not know the state: M = (I + A)^-1 diag(beta).
 // delta_prepare_kernel makes the unit vectors, M, P (the second line's factors), G and E_i = exp(L_7 - L_i) for every block of
 // every request, all blocks at once; delta_scan_kernel walks the blocks: the dots with S, u = M (v - G dots), o, and the update.
+// The unit vectors lie in memory as the walk reads them: two tokens' lanes next to one another, so that one packed multiply-add
+// (fma.rn.f32x2) serves two tokens, and a block's vectors in one run.
 #include "common.cuh"
 
 namespace {
 
 constexpr int BLK = 8;     // tokens a block
 constexpr int COEF = 144;  // floats a (block, head): M [8][8], P [8][8], G [8], E [8]
-constexpr int GROUPS = 16; // groups of threads a CTA of the scan: each owns some neighbouring columns of the state
-constexpr int TPC = 8;     // threads a group: each holds D / 8 rows of the group's columns
+constexpr int R = 16;      // lanes of the scan that share a group of columns of the state: each holds D / 16 rows of them
+constexpr int THREADS = 128;
 
 __device__ __forceinline__ void copy16(float* smem, const float* gmem) {
     const unsigned dst = (unsigned)__cvta_generic_to_shared(smem);
@@ -46,12 +48,27 @@ __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + expf(
 // The index of a request's first block among all blocks of the step: blocks of different requests never share one.
 __device__ __forceinline__ int first_block(int begin, int r) { return begin / BLK + r; }
 
-// grid (blocks of the longest request, G, requests), 128 threads.  y: rows [q: G*D | k: G*D | ...] (pitch ldy), q and k made
-// unit vectors in place.  coef: [blocks, H, COEF]
+// Two tokens at once: a.x * b.x + c.x and a.y * b.y + c.y, each as fmaf would give it.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(d)) : "l"(reinterpret_cast<unsigned long long&>(a)),
+        "l"(reinterpret_cast<unsigned long long&>(b)), "l"(reinterpret_cast<unsigned long long&>(c)));
+    return d;
+}
+
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(d)) : "l"(reinterpret_cast<unsigned long long&>(a)),
+        "l"(reinterpret_cast<unsigned long long&>(b)));
+    return d;
+}
+
+// grid (blocks of the longest request, G, requests), 128 threads.  y: rows [q: G*D | k: G*D | ...] (pitch ldy).
+// units: [blocks, G, 2 (k, q), 4 (pairs of tokens), DS, 2], zeros for missing tokens and for lanes from D on.  coef: [blocks, H, COEF]
 __global__ void __launch_bounds__(128)
-delta_prepare_kernel(float* __restrict__ y, int ldy, const float* __restrict__ b, int ldb, const float* __restrict__ a, int lda,
+delta_prepare_kernel(const float* __restrict__ y, int ldy, const float* __restrict__ b, int ldb, const float* __restrict__ a, int lda,
                      const float* __restrict__ a_log, const float* __restrict__ dt_bias, const int* __restrict__ cu_tokens,
-                     float* __restrict__ coef, int G, int H, int D, float q_scale) {
+                     float* __restrict__ units, float* __restrict__ coef, int G, int H, int D, int DS, float q_scale) {
     extern __shared__ __align__(16) float shared[];
     __shared__ float dots[2][BLK][BLK];  // k_t . k_i and q_t . k_i
     pdl_trigger();
@@ -63,27 +80,38 @@ delta_prepare_kernel(float* __restrict__ y, int ldy, const float* __restrict__ b
     float* sk = shared;              // [8][pitch]
     float* sq = shared + BLK * pitch;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t block = first_block(request, r) + blockIdx.x;
     pdl_wait();
-    for (int t = warp * 2; t < warp * 2 + 2; ++t) {
-        float* qrow = y + (size_t)(begin + t) * ldy + (size_t)g * D;
-        float* krow = qrow + (size_t)G * D;
-        float qq = 0.f, kk = 0.f;
+    {
+        const int t = warp * 2;  // a warp has a pair of tokens
+        const bool has0 = t < count, has1 = t + 1 < count;
+        const float *q0 = y + (size_t)(begin + t) * ldy + (size_t)g * D, *q1 = q0 + ldy, *k0 = q0 + (size_t)G * D, *k1 = q1 + (size_t)G * D;
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
         for (int d = lane; d < D4; d += 32) {
-            const float qv = t < count && d < D ? qrow[d] : 0.f, kv = t < count && d < D ? krow[d] : 0.f;
-            sq[t * pitch + d] = qv;
-            sk[t * pitch + d] = kv;
-            qq = fmaf(qv, qv, qq);
-            kk = fmaf(kv, kv, kk);
+            const float v[4] = {has0 && d < D ? q0[d] : 0.f, has1 && d < D ? q1[d] : 0.f, has0 && d < D ? k0[d] : 0.f, has1 && d < D ? k1[d] : 0.f};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[e] = fmaf(v[e], v[e], s[e]);
+            sq[t * pitch + d] = v[0];
+            sq[(t + 1) * pitch + d] = v[1];
+            sk[t * pitch + d] = v[2];
+            sk[(t + 1) * pitch + d] = v[3];
         }
-        const float fq = q_scale / sqrtf(warp_sum(qq) + 1e-6f), fk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
-        for (int d = lane; d < D; d += 32) {
-            const float qv = sq[t * pitch + d] * fq, kv = sk[t * pitch + d] * fk;
-            sq[t * pitch + d] = qv;
-            sk[t * pitch + d] = kv;
-            if (t < count) {
-                qrow[d] = qv;
-                krow[d] = kv;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[e] = (e < 2 ? q_scale : 1.f) / sqrtf(warp_sum(s[e]) + 1e-6f);
+        float2* uk = reinterpret_cast<float2*>(units + ((block * G + g) * 2 * 4 + warp) * DS * 2);
+        float2* uq = uk + (size_t)4 * DS;
+        for (int d = lane; d < DS; d += 32) {
+            float2 qv = make_float2(0.f, 0.f), kv = qv;
+            if (d < D4) {
+                qv = make_float2(sq[t * pitch + d] * s[0], sq[(t + 1) * pitch + d] * s[1]);
+                kv = make_float2(sk[t * pitch + d] * s[2], sk[(t + 1) * pitch + d] * s[3]);
+                sq[t * pitch + d] = qv.x;
+                sq[(t + 1) * pitch + d] = qv.y;
+                sk[t * pitch + d] = kv.x;
+                sk[(t + 1) * pitch + d] = kv.y;
             }
+            uk[d] = kv;
+            uq[d] = qv;
         }
     }
     __syncthreads();
@@ -124,7 +152,7 @@ delta_prepare_kernel(float* __restrict__ y, int ldy, const float* __restrict__ b
             Ls[t] = __shfl_sync(mask, L, t, 8);
             betas[t] = __shfl_sync(mask, beta, t, 8);
         }
-        float* to = coef + ((size_t)(first_block(request, r) + blockIdx.x) * H + h) * COEF;
+        float* to = coef + (block * H + h) * COEF;
         float T[BLK];  // column j of (I + A)^-1
 #pragma unroll
         for (int t = 0; t < BLK; ++t) {
@@ -140,206 +168,218 @@ delta_prepare_kernel(float* __restrict__ y, int ldy, const float* __restrict__ b
     }
 }
 
-// Eight lanes hold partial sums of eight tokens; they trade halves (4, 2, 1 values) so that lane `sub` ends with token sub's sum.
-__device__ __forceinline__ float trade_sum(const float (&o)[BLK], int sub) {
-    const bool h4 = sub & 4, h2 = sub & 2, h1 = sub & 1;
-    float a[4], b[2];
+// Sixteen lanes hold partial sums of two columns for eight tokens; they trade halves (columns, then tokens) so that lane `sub` ends
+// with the sum of column sub / 8 for token sub % 8.  Every lane has its sums in an order of its own, in which what it keeps stands in
+// front: x[0] is its own column, x[c][u] the pair of tokens u ^ (sub % 8 / 2); so nothing is selected on the way but the last half.
+__device__ __forceinline__ float trade_sum(const float2 (&x)[2][BLK / 2], int sub) {
+    float2 a[4];
 #pragma unroll
-    for (int u = 0; u < 4; ++u) a[u] = (h4 ? o[u + 4] : o[u]) + __shfl_xor_sync(0xffffffffu, h4 ? o[u] : o[u + 4], 4);
+    for (int u = 0; u < 4; ++u) {
+        a[u].x = x[0][u].x + __shfl_xor_sync(0xffffffffu, x[1][u].x, 8);
+        a[u].y = x[0][u].y + __shfl_xor_sync(0xffffffffu, x[1][u].y, 8);
+    }
 #pragma unroll
-    for (int u = 0; u < 2; ++u) b[u] = (h2 ? a[u + 2] : a[u]) + __shfl_xor_sync(0xffffffffu, h2 ? a[u] : a[u + 2], 2);
-    return (h1 ? b[1] : b[0]) + __shfl_xor_sync(0xffffffffu, h1 ? b[0] : b[1], 1);
+    for (int u = 0; u < 2; ++u) {
+        a[u].x += __shfl_xor_sync(0xffffffffu, a[u + 2].x, 4);
+        a[u].y += __shfl_xor_sync(0xffffffffu, a[u + 2].y, 4);
+    }
+    a[0].x += __shfl_xor_sync(0xffffffffu, a[1].x, 2);
+    a[0].y += __shfl_xor_sync(0xffffffffu, a[1].y, 2);
+    return (sub & 1 ? a[0].y : a[0].x) + __shfl_xor_sync(0xffffffffu, sub & 1 ? a[0].x : a[0].y, 1);
 }
 
-// grid (columns of V, H, requests), 128 threads: 16 groups of 8, CPT neighbouring columns a group, DPT rows a thread.
-// q, k, v: columns of y's rows (unit vectors made by the kernel above); coef as above; out: [N, H, V] float32
-template <int DPT, int TB, int CPT>
-__global__ void __launch_bounds__(GROUPS * TPC)
-delta_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, int ld, const float* __restrict__ coef,
-                  float* __restrict__ states, const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, float* __restrict__ out,
-                  int H, int G, int D, int V) {
-    constexpr int COLS = GROUPS * CPT;
-    constexpr int DS = DPT * TPC;   // rows that the CTA's registers have room for (>= D)
-    constexpr int SEG = DPT + 4;    // a part's lanes of a token's q or k, then 4 floats of room: the parts' 16-byte reads fall
-    constexpr int RP = SEG * TPC;   // into different banks; RP: the pitch of a token's row
-    constexpr int NB = TB / BLK;
+// grid (columns of V, H, requests), 128 threads: 8 groups of 16 lanes; a group owns 2 * MC neighbouring columns, a lane DPT rows of
+// them: rows 2 (j * 16 + lane) and the one behind for j < DPT / 2.  Of two neighbouring columns a lane has its own (lane / 8) first,
+// and it takes the block's pairs of tokens in the order u ^ (lane % 8 / 2) (see trade_sum).  units, coef: as above (DS = 16 * DPT); v: [N, H * V] (pitch ld);
+// out: [N, H, V] float32.  NB blocks a stage, the next stage on its way (cp.async) while one is walked.
+template <int DPT, int NB, int MC>
+__global__ void __launch_bounds__(THREADS)
+delta_scan_kernel(const float* __restrict__ units, const float* __restrict__ v, int ld, const float* __restrict__ coef, float* __restrict__ states,
+                  const int* __restrict__ state_slots, const int* __restrict__ cu_tokens, float* __restrict__ out, int H, int G, int D, int V) {
+    constexpr int CPT = 2 * MC, COLS = THREADS / R * CPT, DS = R * DPT, TB = NB * BLK, J = DPT / 2;
+    constexpr int UNITS = 2 * BLK * DS;    // floats a block: k, then q
+    constexpr bool KEEP = DPT <= 8;        // a lane's share of the block's k stays in registers from the dots to the update
     extern __shared__ __align__(16) float shared[];
-    float* sq = shared;                   // [2][TB][RP]
-    float* sk = sq + 2 * TB * RP;         // [2][TB][RP]
-    float* sv = sk + 2 * TB * RP;         // [2][TB][COLS]
-    float* sc = sv + 2 * TB * COLS;       // [2][NB][COEF]
-    float* tile = sc + 2 * NB * COEF;     // [DS][COLS + 1], the state on its way in and out
+    float* su = shared;                    // [2][NB][UNITS]
+    float* sc = su + 2 * NB * UNITS;       // [2][NB][COEF]
+    float* sv = sc + 2 * NB * COEF;        // [2][TB][COLS]
+    float* tile = su;                      // [DS][COLS + 1], the state on its way in and out (before the first and after the last stage)
     pdl_trigger();
     const int r = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * COLS, g = h / (H / G);
-    const int sub = threadIdx.x % TPC, c0 = (threadIdx.x / TPC) * CPT;
-    const int begin = cu_tokens[r], end = cu_tokens[r + 1], slot = state_slots[r], block0 = first_block(begin, r);
+    const int sub = threadIdx.x % R, c0 = (threadIdx.x / R) * CPT;
+    const int col = sub >> 3, tok = sub & 7, turn = tok >> 1;  // what this lane stands for between the sums, and its order of pairs
+    const int begin = cu_tokens[r], end = cu_tokens[r + 1], slot = state_slots[r];
+    const size_t block0 = first_block(begin, r);
     float* state = states + ((size_t)slot * H + h) * D * V;
-    const bool vec = D % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k)) % 16 == 0;
     const bool vec_v = V % 4 == 0 && ld % 4 == 0 && reinterpret_cast<uintptr_t>(v) % 16 == 0 && v0 + COLS <= V;
     pdl_wait();
     if (begin >= end) return;
 
-    auto fetch = [&](int t0, int buf) {
-        const int count = min(TB, end - t0), whole = (count + BLK - 1) / BLK * BLK;
-        if (vec) {
-            const int chunks = D / 4;
-            for (int i = threadIdx.x; i < count * chunks; i += blockDim.x) {
-                const int tt = i / chunks, d = (i % chunks) * 4;
-                const size_t at = ((size_t)buf * TB + tt) * RP + (d / DPT) * SEG + d % DPT;
-                copy16(sq + at, q + (size_t)(t0 + tt) * ld + (size_t)g * D + d);
-                copy16(sk + at, k + (size_t)(t0 + tt) * ld + (size_t)g * D + d);
-            }
-        } else {
-            for (int i = threadIdx.x; i < count * D; i += blockDim.x) {
-                const int tt = i / D, d = i % D;
-                const size_t at = ((size_t)buf * TB + tt) * RP + (d / DPT) * SEG + d % DPT;
-                sq[at] = q[(size_t)(t0 + tt) * ld + (size_t)g * D + d];
-                sk[at] = k[(size_t)(t0 + tt) * ld + (size_t)g * D + d];
-            }
-        }
-        if (vec_v) {
-            for (int i = threadIdx.x; i < count * (COLS / 4); i += blockDim.x) {
-                const int tt = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
-                copy16(sv + ((size_t)buf * TB + tt) * COLS + c, v + (size_t)(t0 + tt) * ld + (size_t)h * V + v0 + c);
-            }
-        } else {
-            for (int i = threadIdx.x; i < count * COLS; i += blockDim.x) {
-                const int tt = i / COLS, c = i % COLS;
-                sv[((size_t)buf * TB + tt) * COLS + c] = v0 + c < V ? v[(size_t)(t0 + tt) * ld + (size_t)h * V + v0 + c] : 0.f;
-            }
-        }
-        const int blocks = whole / BLK;
-        for (int i = threadIdx.x; i < blocks * (COEF / 4); i += blockDim.x) {
-            const int nb = i / (COEF / 4), c = (i % (COEF / 4)) * 4;
-            copy16(sc + ((size_t)buf * NB + nb) * COEF + c, coef + ((size_t)(block0 + (t0 - begin) / BLK + nb) * H + h) * COEF + c);
-        }
-        if (whole > count) {  // a request's last block may hold fewer tokens: zeros in place of the missing ones
-            for (int i = threadIdx.x; i < (whole - count) * RP; i += blockDim.x) {
-                sq[((size_t)buf * TB + count) * RP + i] = 0.f;
-                sk[((size_t)buf * TB + count) * RP + i] = 0.f;
-            }
-            for (int i = threadIdx.x; i < (whole - count) * COLS; i += blockDim.x) sv[((size_t)buf * TB + count) * COLS + i] = 0.f;
-        }
-        asm volatile("cp.async.commit_group;\n" ::);
-    };
-
-    // lanes of q and k beyond D are zeros in both buffers
-    for (int i = threadIdx.x; i < 2 * TB * (DS - D); i += blockDim.x) {
-        const int row = i / (DS - D), d = D + i % (DS - D);
-        const int at = (d / DPT) * SEG + d % DPT;
-        sq[(size_t)row * RP + at] = 0.f;
-        sk[(size_t)row * RP + at] = 0.f;
-    }
-    fetch(begin, 0);
-    for (int i = threadIdx.x; i < D * COLS; i += blockDim.x) {
+    for (int i = threadIdx.x; i < D * COLS; i += THREADS) {
         const int d = i / COLS, c = i % COLS;
         tile[d * (COLS + 1) + c] = v0 + c < V ? state[(size_t)d * V + v0 + c] : 0.f;
     }
     __syncthreads();
-    float S[CPT][DPT];
+    float S[CPT][J][2];
 #pragma unroll
     for (int c = 0; c < CPT; ++c)
 #pragma unroll
-        for (int i = 0; i < DPT; ++i) {
-            const int d = sub * DPT + i;
-            S[c][i] = d < D ? tile[d * (COLS + 1) + c0 + c] : 0.f;
+        for (int j = 0; j < J; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int d = 2 * (j * R + sub) + e;
+                S[c][j][e] = d < D ? tile[d * (COLS + 1) + c0 + (c ^ col)] : 0.f;
+            }
+    __syncthreads();
+
+    auto fetch = [&](int t0, int buf) {
+        const int count = min(TB, end - t0), blocks = (count + BLK - 1) / BLK;
+        const size_t at = block0 + (t0 - begin) / BLK;
+#pragma unroll
+        for (int nb = 0; nb < NB; ++nb) {
+            if (nb >= blocks) break;
+            const float* from = units + ((at + nb) * G + g) * UNITS;
+            float* to = su + (size_t)(buf * NB + nb) * UNITS;
+#pragma unroll
+            for (int i = 0; i < UNITS / 4; i += THREADS)
+                if (UNITS / 4 % THREADS == 0 || i + (int)threadIdx.x < UNITS / 4) copy16(to + (i + threadIdx.x) * 4, from + (i + threadIdx.x) * 4);
+            if (threadIdx.x < COEF / 4) copy16(sc + (size_t)(buf * NB + nb) * COEF + threadIdx.x * 4, coef + ((at + nb) * H + h) * COEF + threadIdx.x * 4);
         }
-    const int live = max(0, min(CPT, V - (v0 + c0)));
+        if (vec_v) {
+            for (int i = threadIdx.x; i < count * (COLS / 4); i += THREADS) {
+                const int tt = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
+                copy16(sv + ((size_t)buf * TB + tt) * COLS + c, v + (size_t)(t0 + tt) * ld + (size_t)h * V + v0 + c);
+            }
+        } else {
+            for (int i = threadIdx.x; i < count * COLS; i += THREADS) {
+                const int tt = i / COLS, c = i % COLS;
+                sv[((size_t)buf * TB + tt) * COLS + c] = v0 + c < V ? v[(size_t)(t0 + tt) * ld + (size_t)h * V + v0 + c] : 0.f;
+            }
+        }
+        for (int i = threadIdx.x; i < (blocks * BLK - count) * COLS; i += THREADS) sv[((size_t)buf * TB + count) * COLS + i] = 0.f;
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+
+    fetch(begin, 0);
     int buf = 0;
     for (int t0 = begin; t0 < end; t0 += TB, buf ^= 1) {
         asm volatile("cp.async.wait_group 0;\n" ::);
         __syncthreads();  // this stage has landed, and everybody has left the other buffer
         if (t0 + TB < end) fetch(t0 + TB, buf ^ 1);
         const int count = min(TB, end - t0);
-        for (int tt = 0; tt < count; tt += BLK) {
-            const float* bq = sq + ((size_t)buf * TB + tt) * RP + sub * SEG;
-            const float* bk = sk + ((size_t)buf * TB + tt) * RP + sub * SEG;
-            const float* bc = sc + ((size_t)buf * NB + tt / BLK) * COEF;
-            // this thread's shares of S^T k and S^T q for the block's tokens
-            float p[CPT][BLK], rd[CPT][BLK];
+#pragma unroll 1
+        for (int nb = 0; nb * BLK < count; ++nb) {
+            const float4* bk = reinterpret_cast<const float4*>(su + (size_t)(buf * NB + nb) * UNITS) + sub;
+            const float4* bq = bk + BLK * DS / 4;
+            const float* bc = sc + (size_t)(buf * NB + nb) * COEF;
+            // this lane's shares of S^T k and S^T q for the block's tokens, two tokens a packed sum
+            float2 p[MC][2][BLK / 2], rd[MC][2][BLK / 2], kk[KEEP ? J : 1][BLK / 2][2];
 #pragma unroll
-            for (int c = 0; c < CPT; ++c)
+            for (int j = 0; j < J; ++j) {
+                float2 ss[CPT][2];
 #pragma unroll
-                for (int u = 0; u < BLK; ++u) p[c][u] = rd[c][u] = 0.f;
+                for (int c = 0; c < CPT; ++c)
 #pragma unroll
-            for (int i = 0; i < DPT; i += 4)
+                    for (int e = 0; e < 2; ++e) ss[c][e] = make_float2(S[c][j][e], S[c][j][e]);
 #pragma unroll
-                for (int u = 0; u < BLK; ++u) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(bk + u * RP + i), q4 = *reinterpret_cast<const float4*>(bq + u * RP + i);
-                    const float kv[4] = {k4.x, k4.y, k4.z, k4.w}, qv[4] = {q4.x, q4.y, q4.z, q4.w};
+                for (int u = 0; u < BLK / 2; ++u) {
+                    // rows 2 (j R + sub), + 1 of tokens 2 (u ^ turn), + 1
+                    const float4 k4 = bk[(u ^ turn) * (DS / 2) + j * R], q4 = bq[(u ^ turn) * (DS / 2) + j * R];
+                    const float2 k2[2] = {make_float2(k4.x, k4.y), make_float2(k4.z, k4.w)}, q2[2] = {make_float2(q4.x, q4.y), make_float2(q4.z, q4.w)};
 #pragma unroll
-                    for (int c = 0; c < CPT; ++c)
+                    for (int e = 0; e < 2; ++e) {
+                        if (KEEP) kk[j][u][e] = k2[e];
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            p[c][u] = fmaf(S[c][i + e], kv[e], p[c][u]);
-                            rd[c][u] = fmaf(S[c][i + e], qv[e], rd[c][u]);
+                        for (int c = 0; c < CPT; ++c) {
+                            float2 &pc = p[c / 2][c % 2][u], &rc = rd[c / 2][c % 2][u];
+                            pc = j == 0 && e == 0 ? mul2(ss[c][e], k2[e]) : fma2(ss[c][e], k2[e], pc);
+                            rc = j == 0 && e == 0 ? mul2(ss[c][e], q2[e]) : fma2(ss[c][e], q2[e], rc);
                         }
+                    }
                 }
-            float Mr[BLK], Pr[BLK], E[BLK];
+            }
+            float Mr[BLK];
+            float2 Pr[BLK / 2], E[BLK / 2];  // in the lane's order of pairs
 #pragma unroll
             for (int i = 0; i < BLK; i += 4) {
-                const float4 m4 = *reinterpret_cast<const float4*>(bc + sub * BLK + i), p4 = *reinterpret_cast<const float4*>(bc + 64 + sub * BLK + i),
-                             e4 = *reinterpret_cast<const float4*>(bc + 136 + i);
+                const float4 m4 = *reinterpret_cast<const float4*>(bc + tok * BLK + i);
                 Mr[i] = m4.x; Mr[i + 1] = m4.y; Mr[i + 2] = m4.z; Mr[i + 3] = m4.w;
-                Pr[i] = p4.x; Pr[i + 1] = p4.y; Pr[i + 2] = p4.z; Pr[i + 3] = p4.w;
-                E[i] = e4.x; E[i + 1] = e4.y; E[i + 2] = e4.z; E[i + 3] = e4.w;
-            }
-            const float gt = bc[128 + sub], gl = bc[128 + BLK - 1];
-            // from here lane `sub` stands for token tt + sub
-            float w[CPT], o[CPT], un[CPT], ue[CPT][BLK];
-#pragma unroll
-            for (int c = 0; c < CPT; ++c) {
-                w[c] = fmaf(-gt, trade_sum(p[c], sub), sv[((size_t)buf * TB + tt + sub) * COLS + c0 + c]);
-                o[c] = gt * trade_sum(rd[c], sub);
-                un[c] = 0.f;
             }
 #pragma unroll
-            for (int i = 0; i < BLK; ++i)
+            for (int u = 0; u < BLK / 2; ++u) {
+                Pr[u] = *reinterpret_cast<const float2*>(bc + 64 + tok * BLK + 2 * (u ^ turn));
+                E[u] = *reinterpret_cast<const float2*>(bc + 136 + 2 * (u ^ turn));
+            }
+            const float gt = bc[128 + tok], gl = bc[128 + BLK - 1];
+            float w[MC], o[MC], un[MC];
+            float2 ue[CPT][BLK / 2];
 #pragma unroll
-                for (int c = 0; c < CPT; ++c) un[c] = fmaf(Mr[i], __shfl_sync(0xffffffffu, w[c], i, TPC), un[c]);
+            for (int m = 0; m < MC; ++m) {
+                w[m] = fmaf(-gt, trade_sum(p[m], sub), sv[((size_t)buf * TB + nb * BLK + tok) * COLS + c0 + 2 * m + col]);
+                float even = 0.f, odd = 0.f;
 #pragma unroll
-            for (int i = 0; i < BLK; ++i)
-#pragma unroll
-                for (int c = 0; c < CPT; ++c) {
-                    const float ui = __shfl_sync(0xffffffffu, un[c], i, TPC);
-                    o[c] = fmaf(Pr[i], ui, o[c]);
-                    ue[c][i] = ui * E[i];
+                for (int i = 0; i < BLK; i += 2) {
+                    even = fmaf(Mr[i], __shfl_sync(0xffffffffu, w[m], i, 8), even);
+                    odd = fmaf(Mr[i + 1], __shfl_sync(0xffffffffu, w[m], i + 1, 8), odd);
                 }
-            if (tt + sub < count) {
-                float* at = out + ((size_t)(t0 + tt + sub) * H + h) * V + v0 + c0;
-                if (CPT == 4 && live == 4 && V % 4 == 0) *reinterpret_cast<float4*>(at) = make_float4(o[0], o[1 % CPT], o[2 % CPT], o[3 % CPT]);
-                else
-#pragma unroll
-                    for (int c = 0; c < CPT; ++c)
-                        if (c < live) at[c] = o[c];
+                un[m] = even + odd;
             }
 #pragma unroll
-            for (int c = 0; c < CPT; ++c)
+            for (int m = 0; m < MC; ++m) o[m] = gt * trade_sum(rd[m], sub);
 #pragma unroll
-                for (int i = 0; i < DPT; ++i) S[c][i] *= gl;
+            for (int u = 0; u < BLK / 2; ++u) {
+                const int from = 2 * (u ^ turn) + (sub & 8);
 #pragma unroll
-            for (int i = 0; i < DPT; i += 4)
-#pragma unroll
-                for (int u = 0; u < BLK; ++u) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(bk + u * RP + i);
-                    const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
-#pragma unroll
-                    for (int c = 0; c < CPT; ++c)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) S[c][i + e] = fmaf(kv[e], ue[c][u], S[c][i + e]);
+                for (int m = 0; m < MC; ++m) {
+                    const float2 mine = make_float2(__shfl_sync(0xffffffffu, un[m], from, 16), __shfl_sync(0xffffffffu, un[m], from + 1, 16));
+                    const float2 other = make_float2(__shfl_sync(0xffffffffu, un[m], from ^ 8, 16), __shfl_sync(0xffffffffu, un[m], (from ^ 8) + 1, 16));
+                    o[m] = fmaf(Pr[u].x, mine.x, o[m]);
+                    o[m] = fmaf(Pr[u].y, mine.y, o[m]);
+                    ue[2 * m][u] = mul2(mine, E[u]);
+                    ue[2 * m + 1][u] = mul2(other, E[u]);
                 }
+            }
+            if (nb * BLK + tok < count) {
+#pragma unroll
+                for (int m = 0; m < MC; ++m)
+                    if (v0 + c0 + 2 * m + col < V) out[((size_t)(t0 + nb * BLK + tok) * H + h) * V + v0 + c0 + 2 * m + col] = o[m];
+            }
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+                float2 k2[BLK / 2][2];
+#pragma unroll
+                for (int u = 0; u < BLK / 2; ++u) {
+                    if (KEEP) { k2[u][0] = kk[j][u][0]; k2[u][1] = kk[j][u][1]; }
+                    else {
+                        const float4 k4 = bk[(u ^ turn) * (DS / 2) + j * R];
+                        k2[u][0] = make_float2(k4.x, k4.y);
+                        k2[u][1] = make_float2(k4.z, k4.w);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < CPT; ++c)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        float2 acc = mul2(k2[0][e], ue[c][0]);
+#pragma unroll
+                        for (int u = 1; u < BLK / 2; ++u) acc = fma2(k2[u][e], ue[c][u], acc);
+                        S[c][j][e] = fmaf(gl, S[c][j][e], acc.x) + acc.y;
+                    }
+            }
         }
     }
     __syncthreads();
 #pragma unroll
     for (int c = 0; c < CPT; ++c)
 #pragma unroll
-        for (int i = 0; i < DPT; ++i) {
-            const int d = sub * DPT + i;
-            if (d < D) tile[d * (COLS + 1) + c0 + c] = S[c][i];
-        }
+        for (int j = 0; j < J; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int d = 2 * (j * R + sub) + e;
+                if (d < D) tile[d * (COLS + 1) + c0 + (c ^ col)] = S[c][j][e];
+            }
     __syncthreads();
-    for (int i = threadIdx.x; i < D * COLS; i += blockDim.x) {
+    for (int i = threadIdx.x; i < D * COLS; i += THREADS) {
         const int d = i / COLS, c = i % COLS;
         if (v0 + c < V) state[(size_t)d * V + v0 + c] = tile[d * (COLS + 1) + c];
     }
@@ -438,32 +478,50 @@ int room(K kernel, size_t smem) {
 
 }  // namespace
 
-// The way for prompts, two launches.  y: [N, >= 2*G*D + H*V] float32 (q and k are left as unit vectors); b, a: [N, H] float32;
-// coef: room for (N / 8 + requests + 1) * H * 144 floats; out: [N, H, V] float32.  wide_columns: 0 = 16 columns of the state a
-// CTA, 1 = as many as the registers take (steps with CTAs enough).
-LLM_EXPORT int llm_delta_scan(float* y, int ldy, const float* b, int ldb, const float* a, int lda, const float* a_log, const float* dt_bias,
-                              float* states, const int* state_slots, const int* cu_tokens, float* coef, float* out, int requests,
-                              int max_query_len, int G, int H, int D, int V, float q_scale, int wide_columns, cudaStream_t stream) {
+// Rows of a head's q or k as the scan has them in memory and in registers: 16 lanes of 2, 4, 8 or 16 rows.
+LLM_EXPORT int llm_delta_rows(int D) { return D <= 32 ? 32 : D <= 64 ? 64 : D <= 128 ? 128 : 256; }
+
+// The way for prompts, two launches.  y: [N, >= 2*G*D + H*V] float32; b, a: [N, H] float32; scratch: room for N / 8 + requests + 1
+// blocks of G * 16 * llm_delta_rows(D) + H * 144 floats; out: [N, H, V] float32.  sms: SMs of the device.
+LLM_EXPORT int llm_delta_scan(const float* y, int ldy, const float* b, int ldb, const float* a, int lda, const float* a_log, const float* dt_bias,
+                              float* states, const int* state_slots, const int* cu_tokens, float* scratch, float* out, int N, int requests,
+                              int max_query_len, int G, int H, int D, int V, float q_scale, int sms, cudaStream_t stream) {
     if (requests <= 0 || max_query_len <= 0) return 0;
-    if (G <= 0 || H <= 0 || H % G || H > 65535 || D <= 0 || D > 256 || V <= 0 || requests > 65535 || ldy < 2 * G * D + H * V || !coef) return LLM_ERR_BAD_ARGUMENT;
-    const int D4 = (D + 3) & ~3;
+    if (G <= 0 || H <= 0 || H % G || H > 65535 || D <= 0 || D > 256 || V <= 0 || requests > 65535 || ldy < 2 * G * D + H * V || !scratch || sms <= 0)
+        return LLM_ERR_BAD_ARGUMENT;
+    const int D4 = (D + 3) & ~3, DS = llm_delta_rows(D);
+    float* units = scratch;
+    float* coef = scratch + (size_t)(N / BLK + requests + 1) * G * 2 * BLK * DS;
     const size_t psmem = (size_t)2 * BLK * (D4 + 4) * sizeof(float);
     int code = launch_pdl(delta_prepare_kernel, dim3((max_query_len + BLK - 1) / BLK, G, requests), dim3(128), psmem, stream, y, ldy, b, ldb, a, lda, a_log,
-                          dt_bias, cu_tokens, coef, G, H, D, q_scale);
+                          dt_bias, cu_tokens, units, coef, G, H, D, DS, q_scale);
     if (code != 0) return code;
-    const float *q = y, *k = y + (size_t)G * D, *v = y + (size_t)2 * G * D;
-    auto go = [&](auto kernel, int dpt, int tb, int cpt) -> int {
-        const int cols = GROUPS * cpt, ds = dpt * TPC;
-        const size_t smem = ((size_t)4 * tb * (dpt + 4) * TPC + (size_t)2 * tb * cols + (size_t)2 * (tb / BLK) * COEF + (size_t)ds * (cols + 1)) * sizeof(float);
+    const float* v = y + (size_t)2 * G * D;
+    auto go = [&](auto kernel, int nb, int mc) -> int {
+        const int cols = THREADS / R * 2 * mc;
+        const dim3 grid((V + cols - 1) / cols, H, requests);
+        size_t smem = ((size_t)2 * nb * (2 * BLK * DS + COEF) + (size_t)2 * nb * BLK * cols) * sizeof(float);
+        const size_t tile = (size_t)DS * (cols + 1) * sizeof(float);
+        if (tile > smem) smem = tile;
+        // A CTA lives as long as the request.  It starts while the last CTAs of the kernel in front still stand on most SMs, and would
+        // crowd onto those that are free first: with few CTAs, each asks for so much shared memory that they spread out evenly.
+        const long long ctas = (long long)grid.x * grid.y * grid.z;
+        for (int per = 1; per <= 3; ++per)
+            if (ctas <= (long long)per * sms) {
+                const size_t want = (size_t)(227 * 1024) / (per + 1) + 1024;
+                if (want > smem) smem = want;
+                break;
+            }
         const int e = room(kernel, smem);
         if (e != 0) return e;
-        return launch_pdl(kernel, dim3((V + cols - 1) / cols, H, requests), dim3(GROUPS * TPC), smem, stream, q, k, v, ldy, (const float*)coef, states,
-                          state_slots, cu_tokens, out, H, G, D, V);
+        return launch_pdl(kernel, grid, dim3(THREADS), smem, stream, (const float*)units, v, ldy, (const float*)coef, states, state_slots, cu_tokens, out,
+                          H, G, D, V);
     };
-    if (D <= 32) return wide_columns ? go(delta_scan_kernel<4, 32, 4>, 4, 32, 4) : go(delta_scan_kernel<4, 32, 1>, 4, 32, 1);
-    if (D <= 64) return wide_columns ? go(delta_scan_kernel<8, 32, 4>, 8, 32, 4) : go(delta_scan_kernel<8, 32, 1>, 8, 32, 1);
-    if (D <= 128) return wide_columns ? go(delta_scan_kernel<16, 16, 2>, 16, 16, 2) : go(delta_scan_kernel<16, 16, 1>, 16, 16, 1);
-    return go(delta_scan_kernel<32, 16, 1>, 32, 16, 1);
+    const bool wide = (long long)((V + 31) / 32) * H * requests >= 2LL * sms;  // CTAs enough when each takes 32 columns of the state
+    if (DS == 32) return wide ? go(delta_scan_kernel<2, 4, 2>, 4, 2) : go(delta_scan_kernel<2, 4, 1>, 4, 1);
+    if (DS == 64) return wide ? go(delta_scan_kernel<4, 4, 2>, 4, 2) : go(delta_scan_kernel<4, 4, 1>, 4, 1);
+    if (DS == 128) return wide ? go(delta_scan_kernel<8, 2, 2>, 2, 2) : go(delta_scan_kernel<8, 2, 1>, 2, 1);
+    return go(delta_scan_kernel<16, 2, 1>, 2, 1);
 }
 
 // The way for few tokens a request, one launch: the recurrence, the norm over each head, its weight [V] and the gate.

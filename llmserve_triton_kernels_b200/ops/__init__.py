@@ -75,7 +75,8 @@ _SIGNATURES = {
     "llm_shift_norm": [_vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "llm_short_conv": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "llm_row_norm": [_vp, _vp, _f, _vp, _vp, _f, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
-    "llm_delta_scan": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
+    "llm_delta_rows": [_i],
+    "llm_delta_scan": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
     "llm_delta_step": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp],
     "llm_row_rmsnorm": [_vp, _i, _i, _vp, _f, _vp, _i, _i, _i, _i, _vp],
     "llm_gated_scan": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _f, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
@@ -1944,8 +1945,7 @@ def delta_rule(y: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: 
         S <- g S        u = b (v - S^T k)        S <- S + k u^T        o = S^T q
 
     and the result is ``o / sqrt(mean(o^2) + eps) * weight * silu(gate)`` over each head's lanes (``weight [value_dim]`` float32,
-    ``gate [N, >= heads * value_dim]`` float32), ``[N, heads * value_dim]`` in ``out_dtype``.  Everything is 32-bit.  ``y`` may be
-    overwritten."""
+    ``gate [N, >= heads * value_dim]`` float32), ``[N, heads * value_dim]`` in ``out_dtype``.  Everything is 32-bit."""
     n = y.shape[0]
     qk, vv = kv_heads * dim, heads * value_dim
     _need(heads % kv_heads == 0 and y.dtype == torch.float32 and y.dim() == 2 and y.stride(1) == 1 and y.shape[1] >= 2 * qk + vv, "delta_rule: y rows hold q, k and v")
@@ -1965,13 +1965,12 @@ def delta_rule(y: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: 
             _check(code, "delta_rule (few tokens)")
             return out
         add_launches(-1)  # a head's state does not fit one CTA: the way for prompts below
-    coef = torch.empty(((n // _DELTA_BLOCK + requests + 1) * heads * _DELTA_COEF,), dtype=torch.float32, device=y.device)
+    blocks, rows = n // _DELTA_BLOCK + requests + 1, library().llm_delta_rows(dim)
+    scratch = torch.empty((blocks * (kv_heads * 2 * _DELTA_BLOCK * rows + heads * _DELTA_COEF),), dtype=torch.float32, device=y.device)
     o = torch.empty((n, heads, value_dim), dtype=torch.float32, device=y.device)
-    cols = 64 if dim <= 64 else 32  # columns of the state a CTA takes where there are CTAs enough
-    wide = -(-value_dim // cols) * heads * requests >= 2 * _sm_count()
     code = _launch("llm_delta_scan", _ptr(y), y.stride(0), _ptr(beta), beta.stride(0), _ptr(decay), decay.stride(0), _ptr(a_log), _ptr(dt_bias), _ptr(states),
-                   _ptr(state_slots), _ptr(ctx.cu_tokens), _ptr(coef), _ptr(o), requests, longest, kv_heads, heads, dim, value_dim, dim ** -0.5,
-                   int(wide), _stream())
+                   _ptr(state_slots), _ptr(ctx.cu_tokens), _ptr(scratch), _ptr(o), n, requests, longest, kv_heads, heads, dim, value_dim, dim ** -0.5,
+                   _sm_count(), _stream())
     add_launches(1)
     _check(code, "delta_rule")
     return head_norm_gate(o, gate[:, :vv], eps, "silu", out_dtype=out_dtype, weight=weight)

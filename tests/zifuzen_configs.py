@@ -54,7 +54,7 @@ ODD = config([
     layer(attention(3, 3, 12, 14, 0.5), moe(10, 3, 7, 1.3, scale=0.8, groups=(2, 1))),
     layer(attention(4, 2, 10, 6, 0.6, kv_from=1), moe(7, 2, 5, 0.8, shared=(8, 2.0))),
     layer(delta(2, 1, 5, 4, 2), moe(8, 4, 6, 1.1, groups=(4, 3), shared=(4, 0.5))),
-], eps=2e-3)
+], eps=5e-2)
 # everything at one or at its end: one head, one tap, one expert a token, groups of one expert, every group kept, one group, an
 # embedding scale of one, no cap
 ONES = config([
