@@ -6,6 +6,8 @@
 
 #include <float.h>
 
+#include <type_traits>
+
 namespace {
 
 // One warp per token.  z: [N, ldz] float32 router logits (the first E of a row; column E, if there is a shared gate,
@@ -135,7 +137,7 @@ router_kernel(const TX* __restrict__ x, int ldx, const float* __restrict__ wr, c
 #pragma unroll
         for (int tt = 0; tt < TT; ++tt) xr[tt] = x + (size_t)min(t0 + tt, N - 1) * ldx;
         if (wide) {
-#pragma unroll(TT == 1 ? 4 : 2)
+#pragma unroll(TT == 1 ? 4 : TT == 2 ? 2 : 1)
             for (int k = lane * 4; k < K; k += 128) {
                 float4 wv[RPW];
                 float xv[TT][4];
@@ -180,6 +182,60 @@ router_kernel(const TX* __restrict__ x, int ldx, const float* __restrict__ wr, c
         float* s = sm + (size_t)TT * rows + (size_t)warp * (2 * E + groups);
         route_row(z + warp * rows, correction, out + (size_t)(t0 + warp) * out_w, s, s + E, E, top, scale, renorm, shared_gate, lane, bias, sigmoid, groups,
                   keep, s + 2 * E);
+    }
+}
+
+// The same for steps of few tokens: one CTA a token, a warp a row of the router matrix at a time.  A warp's first row is on its way
+// before the kernel in front has ended (the weights depend on nothing).  The sums have the order of the kernel above.
+template <typename TX>
+__global__ void __launch_bounds__(1024)
+router_few_kernel(const TX* __restrict__ x, int ldx, const float* __restrict__ wr, const float* __restrict__ correction, float* __restrict__ out,
+                  int K, int E, int top, float scale, int renorm, int shared_gate, const float* __restrict__ bias, int sigmoid, int groups, int keep) {
+    constexpr int AHEAD = 8;  // 16-byte pieces of a row that a lane has in flight
+    extern __shared__ float sm[];  // z[rows], s[E], c[E], and the scores of runs of experts
+    pdl_trigger();
+    const int rows = E + (shared_gate == 1), out_w = E + (shared_gate != 0), t = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const TX* xr = x + (size_t)t * ldx;
+    float4 w[AHEAD];
+    auto ask = [&](int e, int k0) {
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            const int k = k0 + (i * 32 + lane) * 4;
+            w[i] = e < rows && k < K ? *reinterpret_cast<const float4*>(wr + (size_t)e * K + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    };
+    ask(warp, 0);
+    bool waited = false;
+    for (int e = warp; e < rows; e += warps) {
+        float acc = 0.f;
+        for (int k0 = 0; k0 < K; k0 += AHEAD * 128) {
+            if (!waited) pdl_wait();
+            else ask(e, k0);
+            waited = true;
+            float xv[AHEAD][4];
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i) {
+                const int k = k0 + (i * 32 + lane) * 4;
+                xv[i][0] = xv[i][1] = xv[i][2] = xv[i][3] = 0.f;
+                if (k < K) load4(xr + k, xv[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i) {
+                acc = fmaf(w[i].x, xv[i][0], acc);
+                acc = fmaf(w[i].y, xv[i][1], acc);
+                acc = fmaf(w[i].z, xv[i][2], acc);
+                acc = fmaf(w[i].w, xv[i][3], acc);
+            }
+        }
+        acc = warp_sum(acc);
+        if (lane == 0) sm[e] = acc;
+    }
+    if (!waited) pdl_wait();
+    __syncthreads();
+    if (warp == 0) {
+        float* s = sm + rows;
+        route_row(sm, correction, out + (size_t)t * out_w, s, s + E, E, top, scale, renorm, shared_gate, lane, bias, sigmoid, groups, keep, s + 2 * E);
     }
 }
 
@@ -415,12 +471,24 @@ LLM_EXPORT int llm_router(const void* x, int x_dtype, int ldx, const float* wr, 
     if (N <= 0) return 0;
     if (E <= 0 || top < 1 || top > E || E > 2048 || K <= 0 || shared_gate < 0 || shared_gate > 2 ||
         groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups || top > keep * (E / groups)))) return LLM_ERR_BAD_ARGUMENT;
-    // tokens a CTA: one for steps of few tokens (more CTAs, more loads in flight a warp), two otherwise (three CTAs an SM)
-    const int TT = N <= 32 ? 1 : 2;
+    using bf = __nv_bfloat16;
     const int rows_all = E + (shared_gate == 1 ? 1 : 0);  // rows of the router's matrix (2: the last column of out is the constant 1)
+    const size_t align = x_dtype == LLM_F32 ? 16 : 8;
+    if (N <= 32 && K % 4 == 0 && ldx % 4 == 0 && (uintptr_t)wr % 16 == 0 && (uintptr_t)x % align == 0) {
+        const size_t few = ((size_t)rows_all + 2 * E + groups) * sizeof(float);
+        const dim3 block(32 * (rows_all < 32 ? rows_all : 32));
+        if (x_dtype == LLM_F32)
+            return launch_pdl(router_few_kernel<float>, dim3(N), block, few, stream, (const float*)x, ldx, wr, correction, out, K, E, top, scale, renorm,
+                              shared_gate, bias, sigmoid, groups, keep);
+        return launch_pdl(router_few_kernel<bf>, dim3(N), block, few, stream, (const bf*)x, ldx, wr, correction, out, K, E, top, scale, renorm, shared_gate,
+                          bias, sigmoid, groups, keep);
+    }
+    // tokens a CTA: one for steps of few tokens (more CTAs, more loads in flight a warp), two otherwise (three CTAs an SM), eight where
+    // that leaves CTAs enough (the matrix passes through a CTA once for all of its tokens)
+    const int TT = N <= 32 ? 1 : N <= 1184 || E > 512 ? 2 : 8;
     const size_t smem = ((size_t)TT * rows_all + (size_t)TT * (2 * E + groups)) * sizeof(float);
-    const int quads = (rows_all + 3) / 4;  // of rows: a warp each, as far as 16 warps go
-    const dim3 grid((N + TT - 1) / TT), block(32 * (quads < 4 ? 4 : quads > 16 ? 16 : quads));
+    const int quads = (rows_all + 3) / 4, least = TT > 4 ? TT : 4;  // of rows: a warp each, as far as 16 warps go
+    const dim3 grid((N + TT - 1) / TT), block(32 * (quads < least ? least : quads > 16 ? 16 : quads));
     auto go = [&](auto kernel, auto* xp) -> int {
         if (smem > 48 * 1024) {
             const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -428,9 +496,11 @@ LLM_EXPORT int llm_router(const void* x, int x_dtype, int ldx, const float* wr, 
         }
         return launch_pdl(kernel, grid, block, smem, stream, xp, ldx, wr, correction, out, N, K, E, top, scale, renorm, shared_gate, bias, sigmoid, groups, keep);
     };
-    using bf = __nv_bfloat16;
-    if (x_dtype == LLM_F32) return TT == 1 ? go(router_kernel<float, 1>, (const float*)x) : go(router_kernel<float, 2>, (const float*)x);
-    return TT == 1 ? go(router_kernel<bf, 1>, (const bf*)x) : go(router_kernel<bf, 2>, (const bf*)x);
+    auto pick = [&](auto* xp) -> int {
+        using T = std::remove_const_t<std::remove_pointer_t<decltype(xp)>>;
+        return TT == 1 ? go(router_kernel<T, 1>, xp) : TT == 2 ? go(router_kernel<T, 2>, xp) : go(router_kernel<T, 8>, xp);
+    };
+    return x_dtype == LLM_F32 ? pick((const float*)x) : pick((const bf*)x);
 }
 
 LLM_EXPORT int llm_expert_act_scale(const void* x, int ldx, const float* w, int ldw, void* y, int ldy, int dtype, int N, int C, int E,
