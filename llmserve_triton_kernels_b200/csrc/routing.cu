@@ -108,7 +108,7 @@ route_topk_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
 }
 
 // The router's product and the choice in one kernel.  x: [N, K] (any type, read as 32-bit); wr: [E (+ 1), K] float32 (the last
-// row, if there is a shared gate, is the gate's); a CTA takes TT tokens (1 or 2): a warp sums up the logits of four rows at a time for all of
+// row, if there is a shared gate, is the gate's); a CTA takes TT tokens (1, 2 or 8): a warp sums up the logits of four rows at a time for all of
 // them (a lane its share of the elements, then the lanes' sums: the same order whatever else is in the step), then a warp per token
 // chooses.
 template <typename TX, int TT>
